@@ -408,6 +408,8 @@ int lbk_advance_pos(lbk_ctx *ctx, int32_t *pos_dev, void *stream);
  * A step is recorded into a CUDA graph at a cache's first use and replayed afterwards. */
 typedef struct lbk_model lbk_model;
 typedef struct lbk_kv_cache lbk_kv_cache;
+#define LBK_COMPUTE_BF16 0 /* the precisions a family is served in */
+#define LBK_COMPUTE_F32 1  /* everything in 32-bit (families that have it; BitNet does not) */
 typedef struct lbk_model_config {
     size_t hidden_size, intermediate_size, num_attention_heads, num_key_value_heads, num_hidden_layers, vocab_size,
         max_position_embeddings;
@@ -415,6 +417,11 @@ typedef struct lbk_model_config {
     int bos_token_id;
 } lbk_model_config;
 int lbk_model_load(lbk_ctx *ctx, const char *directory, lbk_model **out);
+/* The same with a compute type (lbk_model_load is LBK_COMPUTE_BF16). The family is chosen by the
+ * "architecture" of config.json; files without that key are BitNet's. */
+int lbk_model_load_compute(lbk_ctx *ctx, const char *directory, int compute, lbk_model **out);
+const char *lbk_model_architecture(const lbk_model *model);
+int lbk_model_has_architecture(const char *architecture); /* is the family linked in? */
 /* The same loader for one rank of a tensor-parallel group (the reference has one process and no
  * sharding; its loader is model.rs:149-232). q/k/v/gate/up keep rows [rank*rows/world, ...) of the
  * packed matrix, a contiguous range of the file; o/down keep columns [rank*cols/world, ...), a whole
@@ -455,9 +462,15 @@ int lbk_model_free(lbk_model *model);
 int lbk_model_new_cache(lbk_model *model, size_t batch, size_t capacity, lbk_kv_cache **out);
 size_t lbk_kv_cache_len(const lbk_kv_cache *cache);
 int lbk_kv_cache_reset(lbk_kv_cache *cache);
+/* The same for one sequence of a cache: its positions are given back. */
+int lbk_kv_cache_reset_seq(lbk_kv_cache *cache, size_t seq);
 int lbk_kv_cache_free(lbk_kv_cache *cache);
 int lbk_model_forward(lbk_model *model, lbk_kv_cache *cache, const uint32_t *tokens, size_t n, int all_logits,
                       float *logits_out);
+/* The next n tokens of sequence `seq` of the cache, with the logits of the places want[0 .. n_want) among
+ * them only: logits_out f32 [n_want][vocab] on the host. A portion may be cut anywhere. */
+int lbk_model_forward_rows(lbk_model *model, lbk_kv_cache *cache, size_t seq, const uint32_t *tokens, size_t n, const uint32_t *want,
+                           size_t n_want, float *logits_out);
 int lbk_model_decode(lbk_model *model, lbk_kv_cache *cache, const int32_t *tokens_dev, float *logits_dev,
                      int32_t *next_dev, void *stream);
 /* Rows a prompt pass takes at once (1..8192; default 4096). More rows fill the GEMM's tile rounds

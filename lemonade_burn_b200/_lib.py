@@ -92,6 +92,11 @@ SYMBOLS = [
     ("lbk_tp_gather_f32", _vp, [_vp]),
     ("lbk_tp_argmax", _i, [_vp, _vp, _vp, _sz, _sz, _vp, _vp]),
     ("lbk_model_load", _i, [_vp, C.c_char_p, _pp]),
+    ("lbk_model_load_compute", _i, [_vp, C.c_char_p, _i, _pp]),
+    ("lbk_model_architecture", C.c_char_p, [_vp]),
+    ("lbk_model_has_architecture", _i, [C.c_char_p]),
+    ("lbk_model_forward_rows", _i, [_vp, _vp, _sz, _vp, _sz, _vp, _sz, _vp]),
+    ("lbk_kv_cache_reset_seq", _i, [_vp, _sz]),
     ("lbk_model_load_shard", _i, [_vp, C.c_char_p, _i, _i, _pp]),
     ("lbk_model_load_stats", _i, [_vp, _vp]),
     ("lbk_model_linear", _vp, [_vp, _sz, _i]),

@@ -438,6 +438,7 @@ int attn_tc_init(Ctx *ctx) {
     LBK_CUDA(cudaFuncSetAttribute(attn_prompt_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
     return LBK_OK;
 }
+static const InitHook kInitAttnTc(attn_tc_init);
 
 int launch_attn_prompt_tc(Ctx *ctx, const float *q, const uint16_t *kc, const uint16_t *vc, const int32_t *pos_dev, size_t n, size_t nh, size_t kvh,
                           size_t cap, size_t seq, float *out, cudaStream_t stream) {

@@ -320,6 +320,8 @@ int bf16_init(Ctx *ctx) {
     return LBK_OK;
 }
 
+static const InitHook kInitBf16(bf16_init);
+
 // two token rows and more, rows of whole 16-byte units: the tcgen05 kernel, 64 token rows per pass
 static int launch_bf16_head_tc(Ctx *ctx, const float *x, size_t m, const uint16_t *w, size_t rows, size_t cols, float *out, cudaStream_t stream) {
     HeadParams p{};
@@ -383,3 +385,17 @@ int launch_bf16_linear(Ctx *ctx, const float *x, size_t m, const uint16_t *w, si
 }
 
 }  // namespace lbk
+
+using namespace lbk;
+
+extern "C" {
+
+int lbk_bf16_linear(lbk_ctx *c, const float *x_dev, size_t m, const uint16_t *w_dev, size_t rows, size_t cols,
+                    float *out_dev, void *stream) {
+    if (!c) return fail(LBK_ERR_INVALID, "context is null");
+    if (m * rows && (!out_dev || (cols && (!x_dev || !w_dev)))) return fail(LBK_ERR_INVALID, "lbk_bf16_linear: null buffer");
+    LBK_CUDA(cudaSetDevice(reinterpret_cast<Ctx *>(c)->device));
+    return launch_bf16_linear(reinterpret_cast<Ctx *>(c), x_dev, m, w_dev, rows, cols, out_dev, static_cast<cudaStream_t>(stream));
+}
+
+}  // extern "C"

@@ -493,6 +493,7 @@ int gemm_init(Ctx *ctx) {
     LBK_CUDA(cudaMemset(ctx->gemm_acc, 0, kGemmAccBytes));  // kept zero between launches: the scaling kernel zeroes what it reads
     return LBK_OK;
 }
+static const InitHook kInitGemm(gemm_init);
 
 // Parts to cut every tile's K blocks into. A launch with few tiles against the SM count (small
 // token batches, tensor-parallel shards) or with a ragged last round leaves SMs idle; parts add

@@ -436,6 +436,7 @@ int gemv_init(Ctx *ctx) {
     LBK_CUDA(cudaFuncSetAttribute(gemv_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     return LBK_OK;
 }
+static const InitHook kInitGemv(gemv_init);
 
 int launch_gemv(Ctx *ctx, const GroupArgs &g, cudaStream_t stream) {
     if (g.n < 1 || g.n > LBK_MAX_GROUP) return fail(LBK_ERR_INVALID, "group size %d not in 1..%d", g.n, LBK_MAX_GROUP);

@@ -68,8 +68,12 @@ struct Weight {
 
 int ctx_scratch(Ctx *ctx, size_t bytes, void **out);
 int device_error_status(int word);  // status and message for a non-zero error word
-// One-time per-context kernel attribute set-up (opt-in shared memory sizes).
-int kernels_init(Ctx *ctx);
+// One-time per-context set-up of a kernel file (opt-in shared memory sizes, fixed buffers): lbk_init calls every
+// registered function.
+using InitFn = int (*)(Ctx *ctx);
+struct InitHook {
+    explicit InitHook(InitFn fn);
+};
 int gemv_init(Ctx *ctx);
 int gemm_init(Ctx *ctx);
 int sweep_init(Ctx *ctx);

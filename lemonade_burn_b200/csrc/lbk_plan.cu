@@ -90,15 +90,6 @@ static void plan_build_segments(Plan *p) {
     if (!ok || gi != p->groups.size()) plan_free_segments(p);
 }
 
-int kernels_init(Ctx *ctx) {
-    LBK_TRY(gemv_init(ctx));
-    LBK_TRY(gemm_init(ctx));
-    LBK_TRY(sweep_init(ctx));
-    LBK_TRY(bf16_init(ctx));
-    LBK_TRY(attn_tc_init(ctx));
-    return LBK_OK;
-}
-
 }  // namespace lbk
 
 using namespace lbk;

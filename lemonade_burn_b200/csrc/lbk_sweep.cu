@@ -358,6 +358,7 @@ int sweep_init(Ctx *ctx) {
                                   static_cast<int>(ctx->smem_optin)));
     return LBK_OK;
 }
+static const InitHook kInitSweep(sweep_init);
 
 // Builds the device tables for `groups` (each with m == 1 and f32 input). Returns
 // LBK_ERR_UNSUPPORTED when a group's activation row does not fit the per-warp slice.
