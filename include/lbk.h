@@ -43,6 +43,8 @@ typedef struct lbk_weight lbk_weight; /* a packed ternary matrix resident in dev
 typedef struct lbk_plan lbk_plan;     /* a recorded sequence of fused ternary-linear groups */
 
 #define LBK_MAX_GROUP 4   /* matrices sharing one input in a fused call (q/k/v, gate/up)  */
+#define LBK_COMPUTE_BF16 0 /* the precisions a model family is served in */
+#define LBK_COMPUTE_F32 1 /* everything in 32-bit (families that have it; BitNet does not) */
 #define LBK_GEMV_MAX_M 16 /* token rows served by the bandwidth-bound GEMV kernel         */
 
 /* Message of the last failure on this thread ("" if none). Never NULL. */
@@ -392,7 +394,46 @@ int lbk_argmax(lbk_ctx *ctx, const float *logits_dev, size_t rows, size_t n, int
  * step launched at position >= cap is refused by its kernels (see lbk_check_device_error). */
 int lbk_advance_pos(lbk_ctx *ctx, int32_t *pos_dev, void *stream);
 
+/* ---- bf16-weight layers (no counterpart in the reference, whose projections are ternary) ------------
+ * The mechanisms of the Pefolix family, each callable alone. Row pitches are in values; rows of the compute
+ * type (LBK_COMPUTE_BF16: bf16 bits, LBK_COMPUTE_F32: float) that feed a projection have a pitch of a
+ * multiple of 64 and hold numbers (no NaN) up to it.
+ * lbk_sandwich_norm  x_dev f32 [rows][n]: with y_dev, x += layer_norm(y) * w_post; with w_dev, the rows
+ *                    layer_norm(x) * w go to out_f32 [rows][n] and / or out_bf16 (pitch out_bf16_pitch).
+ *                    layer_norm(x) = (x - mean) / sqrt(var + eps), var = mean of the squared deviations.
+ * lbk_dense_linear   out[t, r] = sum_k x[t, k] * w[r, k], w bf16 [w_rows][w_pitch], zeros past `cols`. gated:
+ *                    w is [gate; up], out = gelu_tanh(gate) * up. relu2: out = max(out, 0)^2. out is the compute
+ *                    type, or f32 with out_f32. experts > 0: w stacks that many matrices of out_rows rows and
+ *                    token rows expert_offs[e] .. expert_offs[e + 1] - 1 belong to expert e (m rows in all).
+ * lbk_attn_window    q [n][heads][dim_pitch], caches [seq][kv_heads][cap][dim_pitch / vdim_pitch] of the compute
+ *                    type (pitches multiples of 16, zeros past dim / vdim). Position i sees j <= i with
+ *                    i - j < window or j < keep_first; score (q . k) * scale, minus 2^(-8 (h + 1) / heads) *
+ *                    (i - j) with distance_bias; softmax. rows_of_seq >= 0: the n rows are positions
+ *                    pos_dev[0] + 0 .. n - 1 of that sequence; -1: row t is sequence t at pos_dev[t], with
+ *                    lbk_attn_window_scratch(n, heads, vdim_pitch) floats of scratch. The keys up to and
+ *                    including each row's own are in the cache already.
+ * lbk_moe_route      softmax over the router logits z [n][z_pitch], the `top` largest and their scores, the
+ *                    tokens sorted by expert: place[t][k] is the sorted row of token t's k-th choice, offs
+ *                    [experts + 1] where each expert starts, sorted_dev (optional) the bf16 rows in that
+ *                    order. scratch_dev: lbk_moe_route_ints(n, experts, top) ints. */
+int lbk_sandwich_norm(lbk_ctx *ctx, float *x_dev, const float *y_dev, const float *w_post_dev, const float *w_dev, size_t rows, size_t n,
+                      float eps, float *out_f32_dev, uint16_t *out_bf16_dev, size_t out_bf16_pitch, void *stream);
+int lbk_dense_linear(lbk_ctx *ctx, int compute, const void *x_dev, size_t x_pitch, size_t m, const uint16_t *w_dev, size_t w_pitch,
+                     size_t w_rows, size_t cols, int gated, size_t out_rows, int relu2, void *out_dev, size_t out_pitch, int out_f32,
+                     const int32_t *expert_offs_dev, size_t experts, void *stream);
+size_t lbk_attn_window_scratch(size_t b, size_t heads, size_t vdim_pitch);
+int lbk_attn_window(lbk_ctx *ctx, int compute, const void *q_dev, const void *kcache_dev, const void *vcache_dev, const int32_t *pos_dev,
+                    size_t n, int rows_of_seq, size_t heads, size_t kv_heads, size_t dim, size_t dim_pitch, size_t vdim, size_t vdim_pitch,
+                    size_t cap, float scale, size_t window, size_t keep_first, int distance_bias, float *scratch_dev, void *out_dev,
+                    size_t out_pitch, void *stream);
+size_t lbk_moe_route_ints(size_t n, size_t experts, size_t top);
+int lbk_moe_route(lbk_ctx *ctx, const float *z_dev, size_t z_pitch, size_t n, size_t experts, size_t top, int32_t *scratch_dev,
+                  const uint16_t *x_dev, size_t x_pitch, uint16_t *sorted_dev, int32_t *ids_out_dev, float *weights_out_dev,
+                  int32_t *place_out_dev, int32_t *offs_out_dev, void *stream);
+
 /* ---- the decoder as a native runtime (crates/lb-model/src/model.rs) ----------------------------
+ * Two families: BitNet (below) and Pefolix (`dir/config.json` with "architecture": "Pefolix" and
+ * `dir/model.safetensors`, bf16 tensors), which has the same calls.
  * lbk_model_load      BitNet::load (model.rs:149-232): `dir/config.json` + `dir/model.lbt.safetensors`
  *                     as lb-convert writes them; the format check and the supported family
  *                     (relu2, tied embeddings) are the reference's; head_dim must be 128.
@@ -408,8 +449,6 @@ int lbk_advance_pos(lbk_ctx *ctx, int32_t *pos_dev, void *stream);
  * A step is recorded into a CUDA graph at a cache's first use and replayed afterwards. */
 typedef struct lbk_model lbk_model;
 typedef struct lbk_kv_cache lbk_kv_cache;
-#define LBK_COMPUTE_BF16 0 /* the precisions a family is served in */
-#define LBK_COMPUTE_F32 1  /* everything in 32-bit (families that have it; BitNet does not) */
 typedef struct lbk_model_config {
     size_t hidden_size, intermediate_size, num_attention_heads, num_key_value_heads, num_hidden_layers, vocab_size,
         max_position_embeddings;

@@ -91,6 +91,12 @@ SYMBOLS = [
     ("lbk_tp_gather_sum", _vp, [_vp]),
     ("lbk_tp_gather_f32", _vp, [_vp]),
     ("lbk_tp_argmax", _i, [_vp, _vp, _vp, _sz, _sz, _vp, _vp]),
+    ("lbk_sandwich_norm", _i, [_vp, _vp, _vp, _vp, _vp, _sz, _sz, _f, _vp, _vp, _sz, _vp]),
+    ("lbk_dense_linear", _i, [_vp, _i, _vp, _sz, _sz, _vp, _sz, _sz, _sz, _i, _sz, _i, _vp, _sz, _i, _vp, _sz, _vp]),
+    ("lbk_attn_window_scratch", _sz, [_sz, _sz, _sz]),
+    ("lbk_attn_window", _i, [_vp, _i, _vp, _vp, _vp, _vp, _sz, _i, _sz, _sz, _sz, _sz, _sz, _sz, _sz, _f, _sz, _sz, _i, _vp, _vp, _sz, _vp]),
+    ("lbk_moe_route_ints", _sz, [_sz, _sz, _sz]),
+    ("lbk_moe_route", _i, [_vp, _vp, _sz, _sz, _sz, _sz, _vp, _vp, _sz, _vp, _vp, _vp, _vp, _vp, _vp]),
     ("lbk_model_load", _i, [_vp, C.c_char_p, _pp]),
     ("lbk_model_load_compute", _i, [_vp, C.c_char_p, _i, _pp]),
     ("lbk_model_architecture", C.c_char_p, [_vp]),
@@ -151,6 +157,14 @@ class LbkError(RuntimeError):
 _lib = None
 
 
+def use(path) -> None:
+    """Load this library instead of liblbk.so (build.library_for: one family's part of it)."""
+    global LIB_PATH
+    if _lib is not None and Path(path) != LIB_PATH:
+        raise RuntimeError(f"{LIB_PATH} is loaded already")
+    LIB_PATH = Path(path)
+
+
 def load() -> C.CDLL:
     """Load liblbk.so and bind every declared symbol. Raises if it is not built."""
     global _lib
@@ -160,7 +174,10 @@ def load() -> C.CDLL:
                 f"{LIB_PATH} is missing: build it with `python -m lemonade_burn_b200.build` "
                 "(there is no CPU fallback)")
         lib = C.CDLL(str(LIB_PATH))
+        whole = LIB_PATH.name == "liblbk.so"
         for name, res, args in SYMBOLS:
+            if not whole and not hasattr(lib, name):  # one family's part of the library
+                continue
             fn = getattr(lib, name)
             fn.restype = res
             fn.argtypes = args

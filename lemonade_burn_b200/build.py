@@ -12,7 +12,15 @@ CSRC = PKG / "csrc"
 LIB = PKG / "liblbk.so"
 OBJ = PKG / "_build"  # object files (git-ignored)
 
-SOURCES = ["lbk_context.cu", "lbk_api.cu", "lbk_gemv.cu", "lbk_quant.cu", "lbk_bf16.cu", "lbk_plan.cu", "lbk_sweep.cu", "lbk_gemm.cu", "lbk_noalloc.cu", "lbk_decoder.cu", "lbk_tp.cu", "lbk_model.cu", "lbk_bitnet.cu", "lbk_convert.cu", "lbk_probe.cu", "lbk_attn_tc.cu"]
+# The runtime every model family needs, and what each family adds. liblbk.so holds all of it; a process that only
+# serves one family can do with that family's part (library_for).
+RUNTIME = ["lbk_context.cu", "lbk_bf16.cu", "lbk_decoder.cu", "lbk_attn_tc.cu", "lbk_model.cu"]
+FAMILIES = {
+    "": ["lbk_api.cu", "lbk_gemv.cu", "lbk_quant.cu", "lbk_plan.cu", "lbk_sweep.cu", "lbk_gemm.cu", "lbk_noalloc.cu", "lbk_tp.cu",
+         "lbk_bitnet.cu", "lbk_convert.cu", "lbk_probe.cu"],
+    "Pefolix": ["lbk_layernorm.cu", "lbk_dense.cu", "lbk_moe.cu", "lbk_attn_window.cu", "lbk_pefolix.cu"],
+}
+SOURCES = RUNTIME + [s for f in FAMILIES.values() for s in f]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC",
@@ -26,10 +34,11 @@ def nvcc_path() -> str:
     raise RuntimeError("nvcc not found; liblbk.so cannot be built")
 
 
-def is_stale() -> bool:
-    if not LIB.exists():
+def is_stale(lib: Path = None) -> bool:
+    lib = lib or LIB
+    if not lib.exists():
         return True
-    t = LIB.stat().st_mtime
+    t = lib.stat().st_mtime
     deps = list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cuh")) + [ROOT / "include" / "lbk.h"]
     return any(d.stat().st_mtime > t for d in deps)
 
@@ -41,11 +50,22 @@ def _run(cmd, env):
     return res.stdout
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every .cu (one object each, side by side, only the ones whose source or any header
-    changed) and link lemonade_burn_b200/liblbk.so. Returns the library path."""
-    if not force and not is_stale():
+def library_for(architecture: str) -> Path:
+    """The library a process that serves this one family loads: liblbk.so when it is built and fresh, else
+    liblbk-<architecture>.so, compiled now from the runtime and the family's own sources."""
+    if not is_stale():
         return LIB
+    if architecture not in FAMILIES or architecture == "":
+        return build()
+    return build(lib=PKG / f"liblbk-{architecture}.so", sources=RUNTIME + FAMILIES[architecture])
+
+
+def build(force: bool = False, verbose: bool = False, lib: Path = None, sources=None) -> Path:
+    """Compile every .cu (one object each, side by side, only the ones whose source or any header
+    changed) and link lemonade_burn_b200/liblbk.so (or `lib` from `sources`). Returns the library path."""
+    lib, sources = lib or LIB, sources or SOURCES
+    if not force and not is_stale(lib):
+        return lib
     from concurrent.futures import ThreadPoolExecutor
     OBJ.mkdir(exist_ok=True)
     env = dict(os.environ)
@@ -55,7 +75,7 @@ def build(force: bool = False, verbose: bool = False) -> Path:
     headers = list(CSRC.glob("*.cuh")) + [ROOT / "include" / "lbk.h"]
     newest_header = max(h.stat().st_mtime for h in headers)
     jobs = []
-    for s in SOURCES:
+    for s in sources:
         src, obj = CSRC / s, OBJ / (Path(s).stem + ".o")
         if force or not obj.exists() or obj.stat().st_mtime < max(src.stat().st_mtime, newest_header):
             cmd = [nvcc, *NVCC_FLAGS, "-c", f"-I{ROOT / 'include'}", f"-I{CSRC}", "-o", str(obj), str(src)]
@@ -66,8 +86,10 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         logs = list(pool.map(lambda c: _run(c, env), jobs))
     if verbose:
         print("\n".join(logs))
-    _run([nvcc, "-shared", "-o", str(LIB)] + [str(OBJ / (Path(s).stem + ".o")) for s in SOURCES], env)
-    return LIB
+    part = lib.with_name(f".{lib.name}.{os.getpid()}")  # a half-written library is never loaded
+    _run([nvcc, "-shared", "-o", str(part)] + [str(OBJ / (Path(s).stem + ".o")) for s in sources], env)
+    os.replace(part, lib)
+    return lib
 
 
 if __name__ == "__main__":

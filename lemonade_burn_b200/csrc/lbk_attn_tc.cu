@@ -31,9 +31,15 @@
 // head: 5e-6 at 2048 keys). What this replaces: the same arithmetic on mma.sync with 16-row tiles
 // per warp (attn_prompt_mma_kernel), which stays for passes of fewer than 64 rows.
 //
+// The windowed form (WINDOW = true; lbk_attn_window.cu says what it computes) is the same kernel with bf16
+// queries in one term, any dim and vdim up to 128, a list of key blocks instead of all of them (the blocks with
+// kept first tokens, then those some row's window reaches), the distance bias taken off the f32 scores, and a
+// bf16 output. A row may see nothing of a block then, so its maximum starts at a finite value.
+//
 // Rows of V past the keys written so far may hold anything (they are multiplied by exact zeros,
 // and 0 * NaN is NaN): the block that reaches past them has them zeroed in shared memory first.
-#include "lbk_internal.cuh"
+#include "lbk_dense.cuh"
+#include "lbk_dense_dev.cuh"
 #include "lbk_ptx.cuh"
 #include "lbk_tcgen05.cuh"
 
@@ -70,14 +76,15 @@ struct AttnParams {
     int n, nh, kvh, cap, seq;
     float scaling;        // log2(e) / sqrt(d)
     int *err_word;
+    // WINDOW
+    const uint16_t *q16;  // [n][nh][dimp]
+    uint16_t *out16;      // [n][nh * vdim], pitch ldo
+    long ldo;
+    int dimp, vdim, vdimp, win, keep;
+    float slope_unit;     // head h: log2(e) * 2^(-8 (h + 1) / nh), or 0
 };
 
-// two f32 -> one word of two bf16 (round to nearest even), `first` in the low half
-__device__ __forceinline__ uint32_t bf16_pair(float first, float second) {
-    uint32_t d;
-    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(d) : "f"(second), "f"(first));
-    return d;
-}
+using dense::bf16_pair;
 // x = hi + lo with hi = bf16(x), lo = bf16(x - hi), for two values at once
 __device__ __forceinline__ void split_pair(float x0, float x1, uint32_t &hi, uint32_t &lo) {
     hi = bf16_pair(x0, x1);
@@ -120,6 +127,7 @@ __device__ __forceinline__ void umma_f16_ts(uint32_t d_tmem, uint32_t a_tmem, ui
                  : "memory");
 }
 
+template <bool WINDOW>
 __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __grid_constant__ AttnParams p) {
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw = ptx::smem_u32(smem_raw);
@@ -163,7 +171,15 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
     const int row0 = tile * kTile;
     const int rows_here = p.n - row0 < kTile ? p.n - row0 : kTile;
     const int written = pos0 + p.n;                          // keys 0 .. written-1 hold numbers
-    const int n_blocks = (pos0 + row0 + rows_here - 1) / kTile + 1;  // key blocks some row of the tile sees
+    // key blocks some row of the tile sees: all of them up to the last row's; with a window those from the first
+    // row's window on (first_blk ..), after the blocks that hold kept tokens in front of it (0 .. kept_blks - 1)
+    int first_blk = 0, kept_blks = 0;
+    if (WINDOW) {
+        first_blk = max(0, pos0 + row0 - p.win + 1) / kTile;
+        kept_blks = min((p.keep + kTile - 1) / kTile, first_blk);
+    }
+    const int n_blocks = kept_blks + (pos0 + row0 + rows_here - 1) / kTile - first_blk + 1;
+    auto block_of = [&](int j) { return WINDOW && j >= kept_blks ? first_blk + j - kept_blks : j; };
     const bool pos_ok = pos0 >= 0 && written <= p.cap;
     if (!pos_ok && tid == 0) atomicExch(p.err_word, 7);
     // the queries of the tile: scaled, as hi + lo, in the K-major SWIZZLE_128B layout (row r of a half
@@ -171,6 +187,15 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
     if (warp < kSoftWarps) {
         const int r = (warp & 3) * 32 + lane;
         const bool live = r < rows_here && pos_ok;
+        if (WINDOW) {
+            const uint16_t *qr = p.q16 + (static_cast<size_t>(row0 + (live ? r : 0)) * p.nh + head) * p.dimp;
+#pragma unroll 4
+            for (int u = (warp >> 2) * 8; u < (warp >> 2) * 8 + 8; ++u) {
+                uint4 a = make_uint4(0u, 0u, 0u, 0u);
+                if (live && u * 8 < p.dimp) a = *reinterpret_cast<const uint4 *>(qr + 8 * u);
+                *reinterpret_cast<uint4 *>(sm + (u >> 3) * kHalf + r * 128 + (((u & 7) ^ (r & 7)) << 4)) = a;
+            }
+        } else {
         const float *qr = p.q + (static_cast<size_t>(row0 + (live ? r : 0)) * p.nh + head) * kHd;
 #pragma unroll 4
         for (int u = (warp >> 2) * 8; u < (warp >> 2) * 8 + 8; ++u) {  // 16-byte unit u of the row: dimensions 8u .. 8u+7; a row's two threads take a half each
@@ -188,6 +213,7 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
             *reinterpret_cast<uint4 *>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
             *reinterpret_cast<uint4 *>(dst + 2 * kHalf) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         }
+        }
         ptx::fence_proxy_async();  // the tensor core reads these through the asynchronous proxy
     }
     tc_fence_before();
@@ -203,15 +229,16 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
         if (lane == 0) {
             int ks = 0, kround = 0;
             for (int j = 0; j < nb; ++j) {
-                const int y = cache_row0 + j * kTile;
+                const int y = cache_row0 + block_of(j) * kTile;
                 if (kround > 0 && !wait_bar(bar(kKEmpty + ks), (kround - 1) & 1, s_abort)) {
                     ok = false;
                     break;
                 }
                 const uint32_t kst = base + kK0 + ks * kBlockBytes;
-                ptx::mbar_arrive_expect_tx(bar(kKFull + ks), kBlockBytes);
+                const bool k2 = !WINDOW || p.dimp > 64, v2 = !WINDOW || p.vdimp > 64;  // a second half of 64 dimensions
+                ptx::mbar_arrive_expect_tx(bar(kKFull + ks), k2 ? kBlockBytes : kHalf);
                 ptx::tma_load_2d(kst, &p.k, bar(kKFull + ks), 0, y);
-                ptx::tma_load_2d(kst + kHalf, &p.k, bar(kKFull + ks), 128, y);
+                if (k2) ptx::tma_load_2d(kst + kHalf, &p.k, bar(kKFull + ks), 128, y);
                 if (++ks == kKStages) {
                     ks = 0;
                     ++kround;
@@ -222,9 +249,9 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
                     break;
                 }
                 const uint32_t vst = base + kV0 + vs * kBlockBytes;
-                ptx::mbar_arrive_expect_tx(bar(kVFull + vs), kBlockBytes);
+                ptx::mbar_arrive_expect_tx(bar(kVFull + vs), v2 ? kBlockBytes : kHalf);
                 ptx::tma_load_2d(vst, &p.v, bar(kVFull + vs), 0, y);
-                ptx::tma_load_2d(vst + kHalf, &p.v, bar(kVFull + vs), 128, y);
+                if (v2) ptx::tma_load_2d(vst + kHalf, &p.v, bar(kVFull + vs), 128, y);
             }
         }
     } else if (warp == kMmaWarp) {
@@ -232,15 +259,18 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
         if (lane == 0 && nb > 0) {
             // D f32, A and B bf16, M = 128, N = 128; for P V the B operand is MN-major (bit 16)
             constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 3) << 17) | ((128u >> 4) << 24);
-            constexpr uint32_t idesc_o = idesc_s | (1u << 16);
+            const uint32_t idesc_o = WINDOW ? ((1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | (static_cast<uint32_t>(p.vdimp >> 3) << 17) | ((128u >> 4) << 24))
+                                            : (idesc_s | (1u << 16));
+            const int dim_steps = WINDOW ? p.dimp >> 4 : 8;
             const uint64_t q_desc = smem_desc_sw128(base);
             int ks = 0, kphase = 0;  // ring position of the K block the next Q K^T reads
             auto issue_s = [&]() {   // S = Qhi K^T + Qlo K^T over the 8 steps of 16 dimensions
                 const uint64_t k_desc = smem_desc_sw128(base + kK0 + ks * kBlockBytes);
 #pragma unroll
-                for (int t = 0; t < 2; ++t)
+                for (int t = 0; t < (WINDOW ? 1 : 2); ++t)
 #pragma unroll
                     for (int st = 0; st < 8; ++st) {
+                        if (WINDOW && st >= dim_steps) break;
                         const uint64_t off = static_cast<uint64_t>((st >> 2) * (kHalf >> 4) + (st & 3) * 2);
                         umma_f16_ss(tmem_base + kColS, q_desc + static_cast<uint64_t>(t * 2 * (kHalf >> 4)) + off, k_desc + off, idesc_s, (t | st) ? 1u : 0u);
                     }
@@ -298,7 +328,8 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
         const int qpos = pos0 + row0 + r;  // the last key this row sees
         const uint32_t lane_field = static_cast<uint32_t>(quad * 32) << 16;
         float *s_pair = reinterpret_cast<float *>(sm + kPairMax);
-        float m = -INFINITY, l = 0.0f;     // m: the maximum the probabilities so far were scaled with; l: this thread's half of the row's sum
+        const float slope = WINDOW && p.slope_unit != 0.0f ? p.slope_unit * exp2f(-8.0f * static_cast<float>(head + 1) / static_cast<float>(p.nh)) : 0.0f;
+        float m = WINDOW ? -1e30f : -INFINITY, l = 0.0f;     // m: the maximum the probabilities so far were scaled with; l: this thread's half of the row's sum
         // a wait whose outcome the whole warp shares: the tensor-memory loads and stores below are warp-wide instructions
         auto wait_all = [&](uint32_t b, uint32_t parity) { return __all_sync(0xffffffffu, wait_bar(b, parity, s_abort)) != 0; };
         auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(1 + quad) : "memory"); };  // the two warps of a quadrant
@@ -316,7 +347,18 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
                 tc_fence_before();
                 __syncwarp();
                 if (lane == 0) ptx::mbar_arrive(bar(kSFree));
-                const int key0 = j * kTile + kh2 * 64;
+                const int key0 = block_of(j) * kTile + kh2 * 64;
+                if (WINDOW) {
+                    const float b0 = slope * static_cast<float>(qpos - key0);
+#pragma unroll
+                    for (int i = 0; i < kTile / 2; ++i)
+                        sv[i] = __float_as_uint(__uint_as_float(sv[i]) * p.scaling - (b0 - slope * static_cast<float>(i)));
+                    if (qpos - key0 >= p.win && key0 + 63 >= p.keep) {  // some of these keys are behind this row's window and not kept
+#pragma unroll
+                        for (int i = 0; i < kTile / 2; ++i)
+                            if (qpos - (key0 + i) >= p.win && key0 + i >= p.keep) sv[i] = 0xff800000u;
+                    }
+                }
                 if (key0 + 63 > qpos) {  // some of these keys are in this row's future
 #pragma unroll
                     for (int i = 0; i < kTile / 2; ++i)
@@ -351,6 +393,7 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
                     l *= corr;
 #pragma unroll 1
                     for (int c = 0; c < 2; ++c) {  // this warp's 64 columns of the output
+                        if (WINDOW && kh2 * 64 + c * 32 >= p.vdimp) break;
                         uint32_t v[32];
                         tmem_ld32(tmem_base + lane_field + kColO + kh2 * 64 + c * 32, v);
                         tmem_ld_wait();
@@ -378,12 +421,13 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
             }
             l += ps0 + ps1;
             // rows of V that no kernel has written: zero them before the tensor core multiplies them by zeros
-            if (j * kTile + kTile > written) {
+            const int blk = block_of(j);
+            if (blk * kTile + kTile > written) {
                 if (!wait_all(bar(kVFull + (j & 1)), (j >> 1) & 1)) {
                     ok = false;
                     continue;
                 }
-                if (j * kTile + r >= written) {  // thread (row r, half kh2) zeroes one 64-dimension half of V row r
+                if (blk * kTile + r >= written) {  // thread (row r, half kh2) zeroes one 64-dimension half of V row r
                     uint8_t *vrow = sm + kV0 + (j & 1) * kBlockBytes + kh2 * kHalf + r * 128;
 #pragma unroll
                     for (int u = 0; u < 8; ++u) *reinterpret_cast<uint4 *>(vrow + u * 16) = make_uint4(0u, 0u, 0u, 0u);
@@ -406,9 +450,34 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
         const float lsum = pair_l[r] + pair_l[kTile + r];
         if (ok && nb > 0) {
             const float inv = 1.0f / lsum;
-            float *dst = p.out + (static_cast<size_t>(row0 + (r < rows_here ? r : 0)) * p.nh + head) * kHd + kh2 * 64;
+            float *dst = WINDOW ? nullptr : p.out + (static_cast<size_t>(row0 + (r < rows_here ? r : 0)) * p.nh + head) * kHd + kh2 * 64;
 #pragma unroll 1
             for (int c = 0; c < 2; ++c) {  // this warp's 64 dimensions of the row
+                if (WINDOW) {
+                    const int d0 = kh2 * 64 + c * 32;
+                    if (d0 >= p.vdimp) break;
+                    uint32_t v[32];
+                    tmem_ld32(tmem_base + lane_field + kColO + d0, v);
+                    tmem_ld_wait();
+                    uint16_t *o = p.out16 + static_cast<size_t>(row0 + r) * p.ldo + static_cast<size_t>(head) * p.vdim + d0;
+                    if (r < rows_here) {
+                        if ((p.vdim & 7) == 0) {
+#pragma unroll
+                            for (int i = 0; i < 32; i += 8)
+                                if (d0 + i < p.vdim) {
+                                    uint32_t w[4];
+#pragma unroll
+                                    for (int e = 0; e < 4; ++e) w[e] = bf16_pair(__uint_as_float(v[i + 2 * e]) * inv, __uint_as_float(v[i + 2 * e + 1]) * inv);
+                                    *reinterpret_cast<uint4 *>(o + i) = make_uint4(w[0], w[1], w[2], w[3]);
+                                }
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 32; ++i)
+                                if (d0 + i < p.vdim) o[i] = dense::f32_bf16(__uint_as_float(v[i]) * inv);
+                        }
+                    }
+                    continue;
+                }
                 uint32_t v[32];
                 tmem_ld32(tmem_base + lane_field + kColO + kh2 * 64 + c * 32, v);
                 tmem_ld_wait();
@@ -435,7 +504,8 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
 
 int attn_tc_init(Ctx *ctx) {
     if (static_cast<size_t>(kSmem) > ctx->smem_optin) return fail(LBK_ERR_UNSUPPORTED, "prompt attention kernel needs %d B of shared memory", kSmem);
-    LBK_CUDA(cudaFuncSetAttribute(attn_prompt_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+    LBK_CUDA(cudaFuncSetAttribute(attn_prompt_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+    LBK_CUDA(cudaFuncSetAttribute(attn_prompt_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
     return LBK_OK;
 }
 static const InitHook kInitAttnTc(attn_tc_init);
@@ -457,7 +527,38 @@ int launch_attn_prompt_tc(Ctx *ctx, const float *q, const uint16_t *kc, const ui
     p.scaling = 1.4426950408889634f / sqrtf(static_cast<float>(kHd));  // scores in units of log 2: the softmax is 2^(s - max)
     p.err_word = ctx->err_word;
     const dim3 grid(static_cast<unsigned>(nh), static_cast<unsigned>((n + kTile - 1) / kTile));
-    LBK_CUDA(launch_chained(attn_prompt_tc_kernel, grid, dim3(kThreads), static_cast<size_t>(kSmem), stream, p));
+    LBK_CUDA(launch_chained(attn_prompt_tc_kernel<false>, grid, dim3(kThreads), static_cast<size_t>(kSmem), stream, p));
+    LBK_CUDA(cudaGetLastError());
+    ctx->launches++;
+    return LBK_OK;
+}
+
+int launch_attn_window_tc(Ctx *ctx, const AttnCall &c, cudaStream_t stream) {
+    if (c.dimp > 128 || c.vdimp > 128 || c.dimp % 16 || c.vdimp % 16 || c.rows_of_seq < 0 || c.ldo % 8)
+        return fail(LBK_ERR_INVALID, "windowed prompt attention: padded head sizes are multiples of 16, at most 128");
+    AttnParams p{};
+    const size_t cache_rows = static_cast<size_t>(c.rows_of_seq + 1) * c.kv_heads * c.cap;
+    LBK_TRY(encode_bytes_map(&p.k, c.kc, c.dimp * 2, cache_rows, c.dimp * 2, 128, kTile));
+    LBK_TRY(encode_bytes_map(&p.v, c.vc, c.vdimp * 2, cache_rows, c.vdimp * 2, 128, kTile));
+    p.pos_dev = c.pos;
+    p.n = static_cast<int>(c.n);
+    p.nh = static_cast<int>(c.heads);
+    p.kvh = static_cast<int>(c.kv_heads);
+    p.cap = static_cast<int>(c.cap);
+    p.seq = c.rows_of_seq;
+    p.scaling = c.scale * 1.4426950408889634f;
+    p.err_word = ctx->err_word;
+    p.q16 = static_cast<const uint16_t *>(c.q);
+    p.out16 = static_cast<uint16_t *>(c.out);
+    p.ldo = c.ldo;
+    p.dimp = static_cast<int>(c.dimp);
+    p.vdim = static_cast<int>(c.vdim);
+    p.vdimp = static_cast<int>(c.vdimp);
+    p.win = c.mask.size;
+    p.keep = c.mask.keep_first;
+    p.slope_unit = c.mask.alibi ? 1.4426950408889634f : 0.0f;
+    const dim3 grid(static_cast<unsigned>(c.heads), static_cast<unsigned>((c.n + kTile - 1) / kTile));
+    LBK_CUDA(launch_chained(attn_prompt_tc_kernel<true>, grid, dim3(kThreads), static_cast<size_t>(kSmem), stream, p));
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;
     return LBK_OK;

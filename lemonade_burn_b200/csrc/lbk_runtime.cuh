@@ -254,6 +254,21 @@ struct Stager {
         }
         return LBK_OK;
     }
+    // `rows` rows of `width` contiguous bytes at data offset `off` -> dst, rows `pitch` bytes apart there
+    int copy_rows(size_t off, size_t rows, size_t width, void *dst, size_t pitch, const char *what) {
+        const size_t rows_per = width ? kStageBytes / width : 0;
+        if (rows_per == 0) return fail(LBK_ERR_UNSUPPORTED, "%s: a row of %zu bytes does not fit the staging buffer", what, width);
+        for (size_t r = 0; r < rows; r += rows_per) {
+            const size_t nr = rows - r < rows_per ? rows - r : rows_per;
+            int s;
+            LBK_TRY(acquire(&s));
+            LBK_TRY(fill(s, data0 + off + r * width, nr * width, what));
+            LBK_CUDA(cudaMemcpy2DAsync(static_cast<char *>(dst) + r * pitch, pitch, buf[s], width, width, nr, cudaMemcpyHostToDevice, st));
+            bytes_to_device += nr * width;
+            LBK_TRY(release(s));
+        }
+        return LBK_OK;
+    }
     // bytes [c0, c0 + width) of each of `rows` rows of pitch `pitch` starting at data offset `off` -> dst (pitch = width)
     int copy_columns(size_t off, size_t rows, size_t pitch, size_t c0, size_t width, void *dst, const char *what) {
         const size_t rows_per = kStageBytes / pitch;

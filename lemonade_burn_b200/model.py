@@ -25,6 +25,7 @@ import torch
 
 from . import _lib, ops
 from .pack import row_bytes
+from .runtime import Batcher, NativeModel, register  # noqa: F401  (Batcher: part of this module's surface)
 from .ternary import Context, default_context
 
 FORMAT = "lemonade-burn-ternary"      # lb-convert/src/lib.rs:14
@@ -331,17 +332,7 @@ def save_checkpoint(directory, cfg: Config, tensors: Dict[str, torch.Tensor]) ->
               metadata={"format": FORMAT, "version": "1", "quant": "absmean-ternary", "layout": "lb-ternary-128x2bit"})
 
 
-class _ModelConfig(C.Structure):
-    _fields_ = [(n, C.c_size_t) for n in ("hidden_size", "intermediate_size", "num_attention_heads", "num_key_value_heads",
-                                          "num_hidden_layers", "vocab_size", "max_position_embeddings")] + \
-               [("rms_norm_eps", C.c_float), ("rope_theta", C.c_float), ("bos_token_id", C.c_int)]
-
-
-class _LoadStats(C.Structure):
-    _fields_ = [("seconds", C.c_double), ("bytes_read", C.c_size_t), ("bytes_to_device", C.c_size_t), ("staging_bytes", C.c_size_t)]
-
-
-class NativeBitNet:
+class NativeBitNet(NativeModel):
     """The same decoder driven entirely by liblbk.so (lbk_model_load / new_cache / forward / decode):
     what a host without a tensor framework binds. Same checkpoint, same kernels, same results as
     `BitNet`; this class only marshals pointers."""
@@ -349,30 +340,20 @@ class NativeBitNet:
     def __init__(self, directory, ctx: Optional[Context] = None, rank: int = 0, world: int = 1):
         """world > 1: this rank's shard only (rows of q/k/v/gate/up, 128-aligned column ranges of
         o/down); such a model serves the tensor-parallel step, not `new_cache` / `forward`."""
-        self.ctx = ctx or default_context()
-        self._lib = self.ctx._lib
         self.rank, self.world = rank, world
-        h = C.c_void_p()
-        if world == 1:
-            _lib.check(self._lib.lbk_model_load(self.ctx.handle, str(directory).encode(), C.byref(h)))
-        else:
-            _lib.check(self._lib.lbk_model_load_shard(self.ctx.handle, str(directory).encode(), rank, world, C.byref(h)))
-        self.handle = h
-        raw = _ModelConfig()
-        _lib.check(self._lib.lbk_model_get_config(h, C.byref(raw)))
+        super().__init__(directory, ctx)
+        raw = self.cfg
         self.cfg = Config(raw.hidden_size, raw.intermediate_size, raw.num_attention_heads, raw.num_key_value_heads,
                           raw.num_hidden_layers, raw.vocab_size, raw.rms_norm_eps, raw.rope_theta, raw.max_position_embeddings,
                           bos_token_id=raw.bos_token_id)
-        self._caches = []
+
+    def _load(self, directory, out) -> int:
+        if self.world == 1:
+            return self._lib.lbk_model_load(self.ctx.handle, str(directory).encode(), out)
+        return self._lib.lbk_model_load_shard(self.ctx.handle, str(directory).encode(), self.rank, self.world, out)
 
     LINEAR_IDS = {"q": 0, "k": 1, "v": 2, "o": 3, "gate": 4, "up": 5, "down": 6}
     NORM_IDS = {"input_norm": 0, "post_attn_norm": 1, "attn_sub_norm": 2, "ffn_sub_norm": 3, "final_norm": 4}
-
-    def load_stats(self) -> dict:
-        """Seconds, bytes read, bytes copied to the device and pinned staging bytes of the load."""
-        s = _LoadStats()
-        _lib.check(self._lib.lbk_model_load_stats(self.handle, C.byref(s)))
-        return {"seconds": s.seconds, "bytes_read": s.bytes_read, "bytes_to_device": s.bytes_to_device, "staging_bytes": s.staging_bytes}
 
     def linear_handle(self, layer: int, name: str) -> int:
         h = self._lib.lbk_model_linear(self.handle, layer, self.LINEAR_IDS[name])
@@ -391,117 +372,5 @@ class NativeBitNet:
     def norm_ptr(self, layer: int, name: str) -> int:
         return int(self._lib.lbk_model_norm(self.handle, layer, self.NORM_IDS[name]))
 
-    def new_cache(self, b: int = 1, cap: int = 0):
-        c = C.c_void_p()
-        _lib.check(self._lib.lbk_model_new_cache(self.handle, b, cap, C.byref(c)))
-        self._caches.append(c)
-        return c
 
-    def cache_len(self, cache) -> int:
-        return int(self._lib.lbk_kv_cache_len(cache))
-
-    def set_prefill_rows(self, rows: int) -> None:
-        """Rows a prompt pass takes at once (default 4096)."""
-        _lib.check(self._lib.lbk_model_set_prefill_rows(self.handle, rows))
-
-    def reset_cache(self, cache) -> None:
-        """Back to an empty sequence; the buffers and the recorded step are kept."""
-        _lib.check(self._lib.lbk_kv_cache_reset(cache))
-
-    def forward(self, tokens, cache, all_logits: bool = False) -> np.ndarray:
-        """model.rs:305: logits [n, vocab] (all_logits) or [vocab] of the last token, on the host."""
-        toks = np.ascontiguousarray(tokens, dtype=np.uint32)
-        out = np.empty((len(toks) if all_logits else 1, self.cfg.vocab_size), dtype=np.float32)
-        _lib.check(self._lib.lbk_model_forward(self.handle, cache, toks.ctypes.data_as(C.c_void_p), len(toks), int(all_logits),
-                                               out.ctypes.data_as(C.c_void_p)))
-        return out if all_logits else out[0]
-
-    def decode(self, tokens_dev: torch.Tensor, cache):
-        """One token per sequence; returns (logits [b, vocab], greedy next tokens [b]) on the device."""
-        b = tokens_dev.shape[0]
-        logits = torch.empty((b, self.cfg.vocab_size), dtype=torch.float32, device=tokens_dev.device)
-        nxt = torch.empty(b, dtype=torch.int32, device=tokens_dev.device)
-        _lib.check(self._lib.lbk_model_decode(self.handle, cache, C.c_void_p(tokens_dev.data_ptr()), C.c_void_p(logits.data_ptr()),
-                                              C.c_void_p(nxt.data_ptr()), C.c_void_p(torch.cuda.current_stream().cuda_stream)))
-        return logits, nxt
-
-    def batcher(self, slots: int, capacity: int = 0) -> "Batcher":
-        return Batcher(self, slots, capacity)
-
-    def close(self):
-        if getattr(self, "handle", None):
-            for bt in list(getattr(self, "_batchers", [])):
-                bt.close()
-            for c in self._caches:
-                self._lib.lbk_kv_cache_free(c)
-            self._caches = []
-            self._lib.lbk_model_free(self.handle)
-            self.handle = None
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass
-
-
-class Batcher:
-    """Continuous batching in front of the batched decode step (lbk_batcher_*): requests queue up, take
-    free slots of one shared cache (prompt pass into the slot), advance together one greedy token per
-    step, and leave as soon as they finish. The reference's server runs its requests one at a time
-    (crates/lb-server/src/main.rs:92-166)."""
-
-    def __init__(self, net: NativeBitNet, slots: int, capacity: int = 0):
-        self.net = net
-        self._lib = net._lib
-        h = C.c_void_p()
-        _lib.check(self._lib.lbk_batcher_create(net.handle, slots, capacity, C.byref(h)))
-        self.handle = h
-        if not hasattr(net, "_batchers"):
-            net._batchers = []
-        net._batchers.append(self)
-
-    def submit(self, prompt, max_new_tokens: int, eos: int = -1) -> int:
-        toks = np.ascontiguousarray(prompt, dtype=np.uint32)
-        rid = C.c_uint64()
-        _lib.check(self._lib.lbk_batcher_submit(self.handle, toks.ctypes.data_as(C.c_void_p), len(toks), max_new_tokens, eos, C.byref(rid)))
-        return int(rid.value)
-
-    def step(self) -> int:
-        """One scheduling step; returns how many requests are still queued or running."""
-        pending = C.c_size_t()
-        _lib.check(self._lib.lbk_batcher_step(self.handle, C.byref(pending)))
-        return int(pending.value)
-
-    def poll(self, rid: int):
-        """(tokens generated so far, finished?)"""
-        n, done = C.c_size_t(), C.c_int()
-        _lib.check(self._lib.lbk_batcher_poll(self.handle, rid, None, 0, C.byref(n), C.byref(done)))
-        out = np.empty(n.value, dtype=np.uint32)
-        _lib.check(self._lib.lbk_batcher_poll(self.handle, rid, out.ctypes.data_as(C.c_void_p), len(out), C.byref(n), C.byref(done)))
-        return out.tolist(), bool(done.value)
-
-    def forget(self, rid: int) -> None:
-        _lib.check(self._lib.lbk_batcher_forget(self.handle, rid))
-
-    def run(self, max_steps: int = 1 << 30) -> int:
-        """Steps until nothing is queued or running; returns the number of steps."""
-        steps = 0
-        while steps < max_steps:
-            steps += 1
-            if self.step() == 0:
-                break
-        return steps
-
-    def close(self):
-        if getattr(self, "handle", None):
-            self._lib.lbk_batcher_destroy(self.handle)
-            self.handle = None
-            if self in getattr(self.net, "_batchers", []):
-                self.net._batchers.remove(self)
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass
+register("", NativeBitNet)
