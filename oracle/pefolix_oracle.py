@@ -1,4 +1,4 @@
-"""Plain numpy restatement of the Pefolix decoder (the checker; float64 by default, nothing shared with the
+"""Plain numpy restatement of the Pefolix decoder (test infrastructure; float64 by default, nothing shared with the
 product path). One function per mechanism, whole sequences at once, no cache:
 
     layer_norm         (x - mean) / sqrt(var + eps) * w, var = mean of the squared deviations

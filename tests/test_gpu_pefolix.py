@@ -1,0 +1,303 @@
+"""The Pefolix family through the runtime (lbk_model_*, lbk_batcher_*) against the plain oracle: whole prompts,
+token by token, portions of any size, several sequences in one cache, slots that are used again, long decoding,
+greedy generation through the batcher. Small configurations of their own, every size different from every other;
+weights whose attention is sharp (large scores), so that one wrong key shows."""
+import json
+
+import numpy as np
+import pytest
+
+pytestmark = pytest.mark.gpu
+
+
+def configs():
+    from lemonade_burn_b200 import pefolix as p
+    a, d, m = p.attention_layer, p.dense_mlp, p.moe_mlp
+    return {
+        # every kind of layer, head sizes that are no multiples of 16, an odd vocabulary
+        "mixed": p.make_config(203, 104, [
+            a(6, 2, 24, 40, 19, 3, 0.9, d(168)),
+            a(4, 4, 32, 16, 7, 0, 0.7, None),
+            a(5, 1, 48, 56, 33, 40, 0.5, m(11, 4, 72, 56)),
+            a(3, 3, 20, 20, None, 0, 0.8, m(6, 1, 40)),
+            a(10, 5, 16, 16, 1, 2, 1.1, m(5, 5, 24, 8))], eps=3e-4),
+        # wide enough for every kernel's tiles and for several 64-key chunks
+        "wide": p.make_config(520, 320, [
+            a(20, 2, 64, 72, 150, 70, 0.4, d(448)),
+            a(8, 1, 128, 128, 64, 1, 0.25, m(24, 6, 160, 200)),
+            a(16, 8, 96, 64, 131, 129, 0.3, d(200))], eps=1e-5),
+        # one head, one key/value head, one expert: values other models make larger
+        "ones": p.make_config(65, 64, [a(1, 1, 64, 64, 8, 1, 1.0, m(1, 1, 64, 64)), a(1, 1, 16, 32, 1000, 0, 1.0, d(16))], eps=1e-6),
+    }
+
+
+TOL = {"float32": 2e-4, "bfloat16": 6e-2}
+
+
+@pytest.fixture(scope="module")
+def nets(ctx, tmp_path_factory):
+    """name -> (config, float64 weights, {dtype: model}), loaded once."""
+    from lemonade_burn_b200 import pefolix, runtime
+    from oracle import pefolix_oracle as po
+    out = {}
+    for i, (name, cfg) in enumerate(configs().items()):
+        d = tmp_path_factory.mktemp(name)
+        pefolix.save_checkpoint(d, cfg, pefolix.random_checkpoint(cfg, 40 + i))
+        _, w = po.load(d)
+        out[name] = (cfg, w, {t: runtime.load_model(d, ctx, t) for t in TOL})
+    return out
+
+
+def tokens(seed, n, vocab):
+    return np.random.default_rng(seed).integers(0, vocab, size=n).astype(np.uint32)
+
+
+def close(got, want, dtype):
+    """Root mean square over the vocabulary (mean taken off), against the spread of the logits."""
+    d = np.asarray(got, dtype=np.float64) - want
+    d -= d.mean(-1, keepdims=True)
+    err = np.atleast_1d(np.sqrt((d * d).mean(-1)) / want.std(-1))
+    if dtype == "bfloat16":
+        # rounding to bf16 turns a close call of a router, or of two keys of a sharp row, now and then (a numpy model
+        # with the same roundings has the same number of such rows): all but a tenth of the rows (a quarter of a few)
+        # have to be close; the 32-bit runs of the same tests have no such allowance
+        spare = len(err) // (10 if len(err) > 40 else 4)
+        assert np.sort(err)[len(err) - 1 - spare] < TOL[dtype] and err.max() < 0.8, (int(err.argmax()), np.sort(err)[-5:])
+    else:
+        assert err.max() < TOL[dtype], (int(err.argmax()), float(err.max()))
+
+
+_memo = {}
+
+
+def logits(nets, name, toks):
+    from oracle import pefolix_oracle as po
+    key = (name, toks.tobytes())
+    if key not in _memo:
+        cfg, w, _ = nets[name]
+        _memo[key] = po.forward(cfg, w, toks)
+    return _memo[key]
+
+
+@pytest.mark.parametrize("dtype", list(TOL))
+@pytest.mark.parametrize("name", ["mixed", "wide", "ones"])
+def test_whole_prompts(nets, name, dtype):
+    cfg, _, models = nets[name]
+    net = models[dtype]
+    assert net.architecture == "Pefolix" and net.cfg.vocab_size == cfg["vocab"] and net.cfg.hidden_size == cfg["width"]
+    for n in (1, 2, 5, 16, 17, 60, 300):
+        t = tokens(n, n, cfg["vocab"])
+        got = net.forward(t, net.new_cache(1, 400), all_logits=True)
+        close(got, logits(nets, name, t), dtype)
+    net.ctx.check_device_error()
+
+
+@pytest.mark.parametrize("dtype", list(TOL))
+@pytest.mark.parametrize("name", ["mixed", "wide", "ones"])
+def test_token_by_token_and_long_decoding(nets, name, dtype):
+    """The recorded decode step from position 0 to 260 (past every window, with kept tokens), and the same tokens as a
+    prompt of 200 followed by single ones."""
+    cfg, _, models = nets[name]
+    net = models[dtype]
+    t = tokens(3, 260, cfg["vocab"])
+    want = logits(nets, name, t)
+    c = net.new_cache(1, 300)
+    close(np.stack([net.forward(t[i:i + 1], c) for i in range(len(t))]), want, dtype)
+    net.reset_cache(c)
+    got = [net.forward(t[:200], c)] + [net.forward(t[i:i + 1], c) for i in range(200, 260)]
+    close(np.stack(got), want[199:], dtype)
+    net.ctx.check_device_error()
+
+
+@pytest.mark.parametrize("dtype", list(TOL))
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+@pytest.mark.parametrize("portions", [[2] * 30, [3, 64, 1, 2, 17, 16, 130, 5, 1, 1, 40], [7, 8, 9, 127, 2, 128]])
+def test_portions(nets, name, dtype, portions):
+    """A prompt in portions gives each position the logits it has in one piece."""
+    cfg, _, models = nets[name]
+    net = models[dtype]
+    n = sum(portions)
+    t = tokens(17, n, cfg["vocab"])
+    c, at, got = net.new_cache(1, n), 0, []
+    for k in portions:
+        got.append(net.forward(t[at:at + k], c, all_logits=True))
+        at += k
+    close(np.concatenate(got), logits(nets, name, t), dtype)
+    net.ctx.check_device_error()
+
+
+@pytest.mark.parametrize("dtype", list(TOL))
+def test_passes_of_a_limited_number_of_rows(nets, dtype):
+    """A prompt longer than a pass goes through in several, the last one ragged; wanted places in any order."""
+    cfg, _, models = nets["mixed"]
+    net = models[dtype]
+    t = tokens(21, 150, cfg["vocab"])
+    want = [149, 0, 64, 63, 65, 128, 2]
+    net.set_prefill_rows(64)
+    try:
+        got = net.forward_rows(t, net.new_cache(1, 150), want)
+    finally:
+        net.set_prefill_rows(4096)
+    close(got, logits(nets, "mixed", t)[want], dtype)
+
+
+@pytest.mark.parametrize("dtype", list(TOL))
+@pytest.mark.parametrize("name", ["mixed", "wide", "ones"])
+def test_unequal_requests_share_a_cache(nets, name, dtype):
+    """Sequences of lengths 1, 37, 90 and 161 in one cache, decoded together, each as if alone; then one of them is
+    given back and another request takes its place while the others go on."""
+    import torch
+    cfg, _, models = nets[name]
+    net = models[dtype]
+    V, lens, more = cfg["vocab"], [1, 37, 90, 161], 12
+    seqs = [tokens(100 + i, n + 2 * more, V) for i, n in enumerate(lens)]
+    c = net.new_cache(4, 220)
+    at = list(lens)
+    for s, n in enumerate(lens):
+        close(net.forward_rows(seqs[s][:n], c, [n - 1], seq=s), logits(nets, name, seqs[s])[n - 1:n], dtype)
+
+    def together(steps):
+        rows = [[] for _ in seqs]
+        for _ in range(steps):
+            tk = torch.tensor([int(seqs[s][at[s]]) for s in range(4)], dtype=torch.int32, device="cuda")
+            lg, _ = net.decode(tk, c)
+            lg = lg.cpu().numpy()
+            for s in range(4):
+                rows[s].append(lg[s])
+                at[s] += 1
+        for s in range(4):
+            close(np.stack(rows[s]), logits(nets, name, seqs[s])[at[s] - steps:at[s]], dtype)
+
+    together(more)
+    seqs[2] = tokens(200, 55 + more, V)
+    net.reset_seq(c, 2)
+    close(net.forward_rows(seqs[2][:55], c, [0, 54], seq=2), logits(nets, name, seqs[2])[[0, 54]], dtype)
+    at[2] = 55
+    together(more)
+    net.ctx.check_device_error()
+
+
+@pytest.mark.parametrize("dtype", list(TOL))
+def test_a_used_cache_is_as_good_as_a_new_one(nets, dtype):
+    """The same request in a fresh cache and in one that a longer request has left: the same bits."""
+    cfg, _, models = nets["wide"]
+    net = models[dtype]
+    t = tokens(5, 180, cfg["vocab"])
+    fresh = net.forward(t, net.new_cache(1, 400), all_logits=True)
+    c = net.new_cache(1, 400)
+    net.forward(tokens(6, 399, cfg["vocab"]), c)
+    net.reset_cache(c)
+    assert np.array_equal(net.forward(t, c, all_logits=True), fresh)
+
+
+def test_one_far_key_decides(nets, tmp_path, ctx):
+    """A model of one layer whose query and key projections single out one token: a request asks for it from just
+    inside and just outside the window and from far behind the kept tokens. In bf16, prompts and decoding."""
+    from lemonade_burn_b200 import pefolix, runtime
+    from oracle import pefolix_oracle as po
+    W, window, keep = 64, 21, 6
+    cfg = pefolix.make_config(80, W, [pefolix.attention_layer(4, 1, 32, 32, window, keep, 1.0, None)], eps=1e-6)
+    t = pefolix.random_checkpoint(cfg, 9)
+    emb = np.zeros((80, W), np.float32)
+    emb[:, :32] = np.random.default_rng(1).standard_normal((80, 32)) * 0.3
+    emb[7, 40], emb[9, 41] = 6.0, 6.0               # token 7 is the key, token 9 asks for it
+    q, k = np.zeros((4 * 32, W), np.float32), np.zeros((32, W), np.float32)
+    for h in range(4):
+        q[h * 32, 41] = 4.0
+    k[0, 40] = 4.0
+    t.update(embed=pefolix.bf16_bits(emb), **{"l0.mix.q": pefolix.bf16_bits(q), "l0.mix.k": pefolix.bf16_bits(k)})
+    pefolix.save_checkpoint(tmp_path, cfg, t)
+    _, w = po.load(tmp_path)
+    net = runtime.load_model(tmp_path, ctx)
+    rng = np.random.default_rng(3)
+    for key_at, ask_at in ((30, 50), (30, 51), (5, 100), (6, 100), (0, 300), (70, 70 + window - 1), (70, 70 + window)):
+        toks = rng.integers(10, 80, size=ask_at + 1).astype(np.uint32)
+        toks[key_at], toks[ask_at] = 7, 9
+        want = po.forward(cfg, w, toks)
+        other = toks.copy()
+        other[key_at] = 33
+        seen = ask_at - key_at < window or key_at < keep
+        moved = np.abs(po.forward(cfg, w, other)[-1] - want[-1]).max() / want[-1].std()
+        assert moved > 0.3 if seen else moved < 1e-6   # the input really asks the question
+        close(net.forward(toks, net.new_cache(1, 310)), want[-1], "bfloat16")
+        c = net.new_cache(1, 310)
+        net.forward(toks[:-1], c)
+        close(net.forward(toks[-1:], c), want[-1], "bfloat16")
+
+
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+def test_greedy_generation(nets, name):
+    """generate() (batcher, prompt passes, recorded steps): in 32-bit the tokens are the oracle's greedy ones; in bf16
+    they do not depend on who shares the batch. More requests than slots, so slots are used again."""
+    from lemonade_burn_b200.generate import generate
+    cfg, w, models = nets[name]
+    from oracle import pefolix_oracle as po
+    prompts = [tokens(300 + i, n, cfg["vocab"]) for i, n in enumerate((1, 9, 40, 3, 70))]
+    new = 10
+    got = generate(models["float32"], prompts, new, slots=2)
+    for p, g in zip(prompts, got):
+        assert len(g) == new
+        lg = po.forward(cfg, w, np.concatenate([p, np.array(g[:-1], dtype=np.uint32)]))[len(p) - 1:]
+        top = np.sort(lg, -1)
+        clear = top[:, -1] - top[:, -2] > 1e-3 * lg.std(-1)
+        assert clear.mean() > 0.7 and (lg.argmax(-1)[clear] == np.array(g)[clear]).all()
+    together = generate(models["bfloat16"], prompts, new, slots=3)
+    alone = [generate(models["bfloat16"], [p], new, slots=3, capacity=90)[0] for p in prompts]
+    same = [a == b for a, b in zip(together, alone)]
+    assert sum(same) >= len(same) - 1, (together, alone)   # another kernel at another batch size may turn one near-tie
+
+
+def test_trace_replay(nets, tmp_path):
+    """The replay program's loop: logits of the wanted places per step, caches taken over by later requests."""
+    from lemonade_burn_b200 import trace
+    cfg, _, models = nets["mixed"]
+    net = models["float32"]
+    a, b = tokens(1, 50, cfg["vocab"]), tokens(2, 33, cfg["vocab"])
+    steps = [("a", a[:20], [0, 19], []), ("a", a[20:22], [], []), ("a", a[22:23], [0], []), ("a", a[23:], [26, 3], ["a"]),
+             ("b", b[:2], [1], []), ("b", b[2:], [30], ["b"])]
+    lines = [json.dumps({"step": i, "entries": [{"id": r, "tokens": [int(x) for x in t], "want": w}], "end": e}) for i, (r, t, w, e) in enumerate(steps)]
+    done = []
+    trace.replay(net, lines, tmp_path, 64, done.append)
+    assert done == list(range(len(steps))) and not (tmp_path / "1.f32").exists()
+    la, lb = logits(nets, "mixed", a), logits(nets, "mixed", b)
+    for i, want in ((0, la[[0, 19]]), (2, la[[22]]), (3, la[[49, 26]]), (4, lb[[1]]), (5, lb[[32]])):
+        close(np.fromfile(tmp_path / f"{i}.f32", dtype="<f4").reshape(-1, cfg["vocab"]), want, "float32")
+
+
+def test_loader_errors(ctx, tmp_path):
+    """A missing tensor, a wrong shape, an unknown mixer, feed-forward or architecture, a truncated file: errors with a
+    message, never a crash; refused calls leave the model usable."""
+    from lemonade_burn_b200 import _lib, pefolix, runtime
+    cfg = pefolix.make_config(40, 32, [pefolix.attention_layer(2, 1, 16, 16, 8, 2, 0.25, pefolix.dense_mlp(24))])
+    t = pefolix.random_checkpoint(cfg, 1)
+
+    def load(c, tensors):
+        pefolix.save_checkpoint(tmp_path, c, tensors)
+        return runtime.NativeModel(tmp_path, ctx)
+
+    net = load(cfg, t)
+    c = net.new_cache(1, 8)
+    with pytest.raises(_lib.LbkError, match="do not fit"):
+        net.forward(np.zeros(9, np.uint32), c)
+    with pytest.raises(_lib.LbkError, match="outside the vocabulary"):
+        net.forward(np.array([40], np.uint32), c)
+    with pytest.raises(_lib.LbkError, match="were asked for"):
+        net.forward_rows(np.zeros(2, np.uint32), c, [2])
+    assert net.forward(np.zeros(8, np.uint32), c).shape == (40,)
+    with pytest.raises(_lib.LbkError, match="l0.mix.v is missing"):
+        load(cfg, {k: v for k, v in t.items() if k != "l0.mix.v"})
+    with pytest.raises(_lib.LbkError, match="l0.mix.k has dtype"):
+        load(cfg, {**t, "l0.mix.k": t["l0.mix.k"][:8]})
+    for edit, text in ((lambda l: l.update(type="other"), "mixer"), (lambda l: l["mlp"].update(kind="other"), "unknown feed-forward"),
+                       (lambda l: l["mixer"].pop("vdim"), "vdim")):
+        bad = json.loads(json.dumps(cfg))
+        edit(bad["layers"][0])
+        with pytest.raises(_lib.LbkError, match=text):
+            load(bad, t)
+    with pytest.raises(_lib.LbkError, match="no model family"):
+        load({**cfg, "architecture": "Other"}, t)
+    net = load(cfg, t)
+    raw = (tmp_path / pefolix.FILE_NAME).read_bytes()
+    (tmp_path / pefolix.FILE_NAME).write_bytes(raw[:-40])
+    with pytest.raises(_lib.LbkError, match="truncated"):
+        runtime.NativeModel(tmp_path, ctx)
