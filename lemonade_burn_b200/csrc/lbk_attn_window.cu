@@ -149,12 +149,14 @@ struct DwLayout {
     }
 };
 
-template <int KS, int VT>  // 16-dimension steps of a key, 8-dimension tiles of a value (upper bounds)
+// KS: 16-dimension steps of a key, VT: 8-dimension tiles of a value; upper bounds, or (EXACT) the sizes themselves
+template <int KS, int VT, bool EXACT>
 __global__ void __launch_bounds__(kDwWarps * 32) attn_window_decode_kernel(const WinParams p) {
     ptx::pdl_trigger();
     ptx::pdl_wait();
     extern __shared__ __align__(16) uint8_t dw_smem[];
-    const DwLayout L(p.dimp, p.vdimp);
+    const int dimp = EXACT ? KS * 16 : p.dimp, vdimp = EXACT ? VT * 8 : p.vdimp;
+    const DwLayout L(dimp, vdimp);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int group = p.heads / p.kv_heads, htiles = (group + 15) / 16;
     const int sp = blockIdx.x, kh = blockIdx.y / htiles, h0 = (blockIdx.y % htiles) * 16, b = blockIdx.z;
@@ -167,13 +169,13 @@ __global__ void __launch_bounds__(kDwWarps * 32) attn_window_decode_kernel(const
     const Visible vis(p, pos);
     const int per = ((vis.total + p.splits - 1) / p.splits + kDwKeys - 1) / kDwKeys * kDwKeys;
     const int u0 = min(vis.total, sp * per), u1 = min(vis.total, u0 + per);
-    const uint16_t *kb = static_cast<const uint16_t *>(p.kc) + (static_cast<size_t>(b) * p.kv_heads + kh) * p.cap * p.dimp;
-    const uint16_t *vb = static_cast<const uint16_t *>(p.vc) + (static_cast<size_t>(b) * p.kv_heads + kh) * p.cap * p.vdimp;
-    const int ku = p.dimp / 8, vu = p.vdimp / 8;                  // 16-byte units per row
+    const uint16_t *kb = static_cast<const uint16_t *>(p.kc) + (static_cast<size_t>(b) * p.kv_heads + kh) * p.cap * dimp;
+    const uint16_t *vb = static_cast<const uint16_t *>(p.vc) + (static_cast<size_t>(b) * p.kv_heads + kh) * p.cap * vdimp;
+    const int ku = dimp / 8, vu = vdimp / 8;                  // 16-byte units per row
     for (int i = tid; i < 16 * ku; i += kDwWarps * 32) {
         const int r = i / ku, c = i - r * ku;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (r < nh) v = *reinterpret_cast<const uint4 *>(static_cast<const uint16_t *>(p.q) + (static_cast<size_t>(b) * p.heads + head0 + r) * p.dimp + c * 8);
+        if (r < nh) v = *reinterpret_cast<const uint4 *>(static_cast<const uint16_t *>(p.q) + (static_cast<size_t>(b) * p.heads + head0 + r) * dimp + c * 8);
         *reinterpret_cast<uint4 *>(dw_smem + L.q + r * L.krow + c * 16) = v;
     }
     auto stage = [&](int buf, int uc) {
@@ -184,7 +186,7 @@ __global__ void __launch_bounds__(kDwWarps * 32) attn_window_decode_kernel(const
             uint8_t *dst = c < ku ? dk + r * L.krow + c * 16 : dv + r * L.vrow + (c - ku) * 16;
             if (r < cnt) {
                 const int key = vis.key(uc + r);
-                ptx::cp_async_16(ptx::smem_u32(dst), c < ku ? kb + static_cast<size_t>(key) * p.dimp + c * 8 : vb + static_cast<size_t>(key) * p.vdimp + (c - ku) * 8);
+                ptx::cp_async_16(ptx::smem_u32(dst), c < ku ? kb + static_cast<size_t>(key) * dimp + c * 8 : vb + static_cast<size_t>(key) * vdimp + (c - ku) * 8);
             } else {
                 *reinterpret_cast<uint4 *>(dst) = make_uint4(0u, 0u, 0u, 0u);  // weight zero, but the bits must be numbers
             }
@@ -195,7 +197,7 @@ __global__ void __launch_bounds__(kDwWarps * 32) attn_window_decode_kernel(const
     const uint32_t k_lane0 = ptx::smem_u32(dw_smem) + (warp * 16 + (lane & 7)) * L.krow + (lane >> 3) * 16;
     const uint32_t v_lane0 = ptx::smem_u32(dw_smem) + kDwKeys * L.krow + (warp * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * L.vrow + (lane >> 4) * 16;
     const float sl0 = head_slope(p, head0 + g), sl1 = head_slope(p, head0 + g + 8);
-    const int ks_n = p.dimp / 16, vp_n = p.vdimp / 16;
+    const int ks_n = dimp / 16, vp_n = vdimp / 16;
     float o[VT][4];
 #pragma unroll
     for (int j = 0; j < VT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
@@ -288,7 +290,7 @@ __global__ void __launch_bounds__(kDwWarps * 32) attn_window_decode_kernel(const
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     __syncthreads();  // the stages are free: [warp][16 heads][vdimp + 4] floats
     float *s_o = reinterpret_cast<float *>(dw_smem);
-    const int mrow = p.vdimp + 4;
+    const int mrow = vdimp + 4;
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         float *r = s_o + (warp * 16 + g + 8 * h) * mrow;
@@ -296,25 +298,25 @@ __global__ void __launch_bounds__(kDwWarps * 32) attn_window_decode_kernel(const
         for (int j = 0; j < VT; ++j)
             if (j < 2 * vp_n) *reinterpret_cast<float2 *>(r + 8 * j + 2 * t) = make_float2(o[j][2 * h], o[j][2 * h + 1]);
         if (t == 0) {
-            r[p.vdimp] = h ? m1 : m0;
-            r[p.vdimp + 1] = h ? l1 : l0;
+            r[vdimp] = h ? m1 : m0;
+            r[vdimp + 1] = h ? l1 : l0;
         }
     }
     __syncthreads();
-    const int prow = p.vdimp + 4;
-    for (int i = tid; i < nh * (p.vdimp / 4); i += kDwWarps * 32) {
-        const int r = i / (p.vdimp / 4), d = (i - r * (p.vdimp / 4)) * 4;
+    const int prow = vdimp + 4;
+    for (int i = tid; i < nh * (vdimp / 4); i += kDwWarps * 32) {
+        const int r = i / (vdimp / 4), d = (i - r * (vdimp / 4)) * 4;
         float gm = -INFINITY;
 #pragma unroll
-        for (int w = 0; w < kDwWarps; ++w) gm = fmaxf(gm, s_o[(w * 16 + r) * mrow + p.vdimp]);
+        for (int w = 0; w < kDwWarps; ++w) gm = fmaxf(gm, s_o[(w * 16 + r) * mrow + vdimp]);
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
         float sum = 0.0f;
 #pragma unroll
         for (int w = 0; w < kDwWarps; ++w) {
             const float *x = s_o + (w * 16 + r) * mrow;
-            const float wm = x[p.vdimp];
+            const float wm = x[vdimp];
             const float wt = wm == -INFINITY ? 0.0f : __expf(wm - gm);
-            sum += wt * x[p.vdimp + 1];
+            sum += wt * x[vdimp + 1];
             a.x += wt * x[d]; a.y += wt * x[d + 1]; a.z += wt * x[d + 2]; a.w += wt * x[d + 3];
         }
         if (p.splits == 1) {
@@ -327,8 +329,8 @@ __global__ void __launch_bounds__(kDwWarps * 32) attn_window_decode_kernel(const
             float *dst = p.part + ((static_cast<size_t>(b) * p.heads + head0 + r) * p.splits + sp) * prow;
             *reinterpret_cast<float4 *>(dst + d) = a;
             if (d == 0) {
-                dst[p.vdimp] = gm;  // -inf for an empty slice: the merge gives it no weight
-                dst[p.vdimp + 1] = sum;
+                dst[vdimp] = gm;  // -inf for an empty slice: the merge gives it no weight
+                dst[vdimp + 1] = sum;
             }
         }
     }
@@ -383,9 +385,11 @@ int launch_generic(Ctx *ctx, const WinParams &p, cudaStream_t st) {
 
 int attn_window_init(Ctx *) {
     const DwLayout small(64, 64), mid(128, 128), big(256, 256);
-    LBK_CUDA(cudaFuncSetAttribute(attn_window_decode_kernel<4, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, small.total));
-    LBK_CUDA(cudaFuncSetAttribute(attn_window_decode_kernel<8, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, mid.total));
-    LBK_CUDA(cudaFuncSetAttribute(attn_window_decode_kernel<16, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, big.total));
+    LBK_CUDA(cudaFuncSetAttribute(attn_window_decode_kernel<4, 8, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, small.total));
+    LBK_CUDA(cudaFuncSetAttribute(attn_window_decode_kernel<8, 16, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, mid.total));
+    LBK_CUDA(cudaFuncSetAttribute(attn_window_decode_kernel<16, 32, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big.total));
+    LBK_CUDA(cudaFuncSetAttribute(attn_window_decode_kernel<4, 8, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, small.total));
+    LBK_CUDA(cudaFuncSetAttribute(attn_window_decode_kernel<8, 16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, mid.total));
     return LBK_OK;
 }
 const InitHook kInitAttnWindow(attn_window_init);
@@ -448,7 +452,9 @@ int launch_attn_window(Ctx *ctx, const AttnCall &c, cudaStream_t st) {
     p.part = c.scratch;
     const dim3 grid(static_cast<unsigned>(splits), static_cast<unsigned>(tiles), static_cast<unsigned>(c.n));
     const size_t smem = static_cast<size_t>(DwLayout(p.dimp, p.vdimp).total);
-    void (*k)(WinParams) = dmax <= 64 ? attn_window_decode_kernel<4, 8> : dmax <= 128 ? attn_window_decode_kernel<8, 16> : attn_window_decode_kernel<16, 32>;
+    void (*k)(WinParams) = dmax <= 64 ? attn_window_decode_kernel<4, 8, false> : dmax <= 128 ? attn_window_decode_kernel<8, 16, false> : attn_window_decode_kernel<16, 32, false>;
+    if (p.dimp == 64 && p.vdimp == 64) k = attn_window_decode_kernel<4, 8, true>;
+    if (p.dimp == 128 && p.vdimp == 128) k = attn_window_decode_kernel<8, 16, true>;
     LBK_CUDA(launch_chained(k, grid, dim3(kDwWarps * 32), smem, st, p));
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;

@@ -159,6 +159,7 @@ int lbk_destroy(lbk_ctx *c) {
     if (ctx->small_scratch) cudaFree(ctx->small_scratch);
     if (ctx->gemm_acc) cudaFree(ctx->gemm_acc);
     if (ctx->bf16_x) cudaFree(ctx->bf16_x);
+    if (ctx->few_parts) cudaFree(ctx->few_parts);
     if (ctx->own_stream) cudaStreamDestroy(ctx->own_stream);
     delete ctx;
     return LBK_OK;

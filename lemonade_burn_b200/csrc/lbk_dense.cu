@@ -7,13 +7,18 @@
 //                      is two MMAs' operands as it is (the contraction index may be permuted as long as both
 //                      operands are permuted alike), so weights go global -> registers -> tensor core without
 //                      shared memory or shuffles. The 16 warps of a CTA split K and meet in shared memory once per
-//                      tile. The norms in front of the projection run in the prologue (at one or two tokens),
+//                      tile. Where whole tiles would leave SMs idle in the last round, the (tile, K) stream is cut into
+//                      equal runs instead: a tile shared by several CTAs leaves partial sums in memory, and the one
+//                      that arrives last adds them up in CTA order. The norms in front of the projection run in the prologue (at one or two tokens),
 //                      while the CTA's first weight rows are on their way to L2.
 //   dense_gemm_kernel  more tokens: tcgen05 (kind::f16), 128 weight rows x up to 256 tokens a tile, both operands
 //                      by TMA (SWIZZLE_128B, 64 columns a stage), two accumulators in tensor memory so that the
 //                      epilogue of one tile runs under the MMAs of the next, one persistent CTA per SM. A gated
 //                      projection keeps gate and up accumulators of the same 128 rows side by side, so the
-//                      product is taken where both sit in one thread's registers. With experts the tokens
+//                      product is taken where both sit in one thread's registers. Few tiles and a long K (a short
+//                      portion of a prompt) are cut along K over a cluster of 2 to 8 CTAs, whose accumulators meet
+//                      in shared memory: every CTA reads its share of the tokens from all of them, in rank order.
+//                      With experts the tokens
 //                      arrive sorted and the tile list comes from the device-side counts.
 //   dense_f32_kernel   everything in 32-bit (FMA), for LBK_COMPUTE_F32.
 #include "lbk_dense.cuh"
@@ -29,9 +34,12 @@ using namespace tc;
 
 // ---- few tokens ---------------------------------------------------------------------------------
 constexpr int kFewThreads = 512, kFewWarps = 16;
-constexpr int kFewUnroll = 4;               // 32-column chunks in flight per warp
 constexpr int kFewPreMax = 2;               // tokens whose norms run in the prologue
 constexpr size_t kFewXSmem = 96 * 1024;     // activations in shared memory up to this, else read through L1
+
+constexpr int kFewPart = 2 * 2 * 128;       // floats of a partial tile: gate and up, 16 tokens, 16 rows
+constexpr int kFewMaxTiles = 1 << 14, kFewMaxCtas = 512;
+constexpr int kFewPrefetch = 2;             // 128-byte lines a thread asks L2 for ahead of the kernel in front
 
 struct FewParams {
     const uint16_t *w;
@@ -40,6 +48,9 @@ struct FewParams {
     const uint16_t *x;
     long ldx;
     int x_smem, xs_stride;                  // bytes per token row in shared memory
+    int per;                                // 32-column chunks of the (tile, K) stream a CTA takes
+    float *parts;                           // [2 * CTAs][kFewPart] partial sums of tiles shared between CTAs
+    int *counters;                          // [tiles], zero at rest
     DenseEpi epi;
     DensePre pre;
     int n;                                  // columns of the normed row
@@ -122,15 +133,22 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
     uint8_t *s_x = few_smem + 2 * kFewWarps * kPart * sizeof(float);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     ptx::pdl_trigger();
-    // the weights are constants: this CTA's first tile starts moving to L2 while the kernel in front finishes
-    if (static_cast<int>(blockIdx.x) < p.tiles) {
-        const int lines = p.chunks / 2;     // 128-byte lines of a row (pitch is a multiple of 64 columns)
+    const int s_begin = static_cast<int>(blockIdx.x) * p.per, s_end = min(p.tiles * p.chunks, s_begin + p.per);
+    // the weights are constants: the first of this CTA's rows start moving to L2 while the kernel in front finishes
+    {
+        int at = s_begin, left = kFewPrefetch * kFewThreads;
+        while (at < s_end && left > 0) {
+            const int tile = at / p.chunks, a = at - tile * p.chunks, b = min(p.chunks, a + s_end - at);
+            const int l0 = a / 2, lines = (b + 1) / 2 - l0;  // 128-byte lines of a row (pitch is a multiple of 64 columns)
 #pragma unroll
-        for (int a = 0; a < NA; ++a)
-            for (int i = tid; i < 16 * lines; i += kFewThreads) {
-                const int r = min(static_cast<int>(blockIdx.x) * 16 + i / lines, p.out_rows - 1) + a * p.up_row;
-                asm volatile("prefetch.global.L2 [%0];" ::"l"(p.w + static_cast<size_t>(r) * p.pitch + (i % lines) * 64));
-            }
+            for (int w = 0; w < NA; ++w)
+                for (int i = tid; i < 16 * lines; i += kFewThreads) {
+                    const int r = min(tile * 16 + i / lines, p.out_rows - 1) + w * p.up_row;
+                    asm volatile("prefetch.global.L2 [%0];" ::"l"(p.w + static_cast<size_t>(r) * p.pitch + (l0 + i % lines) * 64));
+                }
+            left -= NA * 16 * lines;
+            at += b - a;
+        }
     }
     ptx::pdl_wait();
     int pos0;
@@ -146,49 +164,90 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
         }
         __syncthreads();
     }
-    const int c_per = (p.chunks + kFewWarps - 1) / kFewWarps;
-    const int c0 = min(p.chunks, warp * c_per), c1 = min(p.chunks, c0 + c_per);
-    int buf = 0;
-    for (int tile = blockIdx.x; tile < p.tiles; tile += gridDim.x, buf ^= 1) {
-        float acc[NA][NTL][4];
-#pragma unroll
-        for (int a = 0; a < NA; ++a)
-#pragma unroll
-            for (int j = 0; j < NTL; ++j) acc[a][j][0] = acc[a][j][1] = acc[a][j][2] = acc[a][j][3] = 0.0f;
-        const int r_lo = min(tile * 16 + g, p.out_rows - 1), r_hi = min(tile * 16 + g + 8, p.out_rows - 1);
-        const uint16_t *w_lo = p.w + static_cast<size_t>(r_lo) * p.pitch + t * 8, *w_hi = p.w + static_cast<size_t>(r_hi) * p.pitch + t * 8;
+    __shared__ int s_last;
+    // The CTA's run of the stream is a sequence of tile parts, a warp's share of one part a sequence of steps of U
+    // chunks. The loads of a step are issued one step ahead, across tiles too: a warp always has two steps in flight.
+    constexpr int U = DUAL ? 2 : 4;
+    struct Step {
+        int tile, k0, k1, c, c1;
+    };
+    int at = s_begin;
+    auto next_part = [&](Step &q) {
+        q.tile = at / p.chunks;
+        q.k0 = at - q.tile * p.chunks;
+        q.k1 = min(p.chunks, q.k0 + s_end - at);
+        at += q.k1 - q.k0;
+        const int c_per = (q.k1 - q.k0 + kFewWarps - 1) / kFewWarps;
+        q.c = min(q.k1, q.k0 + warp * c_per);
+        q.c1 = min(q.k1, q.c + c_per);
+    };
+    uint4 wl[NA][U], wh[NA][U], nl[NA][U], nh[NA][U];
+    auto load = [&](const Step &q, uint4 (&lo)[NA][U], uint4 (&hi)[NA][U]) {
+        const uint16_t *a = p.w + static_cast<size_t>(min(q.tile * 16 + g, p.out_rows - 1)) * p.pitch + t * 8;
+        const uint16_t *b = p.w + static_cast<size_t>(min(q.tile * 16 + g + 8, p.out_rows - 1)) * p.pitch + t * 8;
         const size_t up = static_cast<size_t>(p.up_row) * p.pitch;
-        for (int c = c0; c < c1; c += kFewUnroll) {
-            uint4 wl[NA][kFewUnroll], wh[NA][kFewUnroll];
 #pragma unroll
-            for (int i = 0; i < kFewUnroll; ++i)
-                if (c + i < c1) {
+        for (int i = 0; i < U; ++i)
+            if (q.c + i < q.c1) {
+#pragma unroll
+                for (int w = 0; w < NA; ++w) {
+                    lo[w][i] = __ldcs(reinterpret_cast<const uint4 *>(a + w * up + (q.c + i) * 32));
+                    hi[w][i] = __ldcs(reinterpret_cast<const uint4 *>(b + w * up + (q.c + i) * 32));
+                }
+            }
+    };
+    float acc[NA][NTL][4];
+#pragma unroll
+    for (int a = 0; a < NA; ++a)
+#pragma unroll
+        for (int j = 0; j < NTL; ++j) acc[a][j][0] = acc[a][j][1] = acc[a][j][2] = acc[a][j][3] = 0.0f;
+    int buf = 0;
+    Step cur, nxt;
+    bool more = at < s_end;
+    if (more) {
+        next_part(cur);
+        load(cur, wl, wh);
+    }
+    while (more) {
+        nxt = cur;
+        const bool part_done = cur.c + U >= cur.c1;
+        if (!part_done) {
+            nxt.c += U;
+        } else if (at < s_end) {
+            next_part(nxt);
+        } else {
+            more = false;
+        }
+        if (more) load(nxt, nl, nh);
+#pragma unroll
+        for (int i = 0; i < U; ++i)
+            if (cur.c + i < cur.c1) {
+#pragma unroll
+                for (int j = 0; j < NTL; ++j) {
+                    uint4 b = make_uint4(0u, 0u, 0u, 0u);
+                    const int tk = j * 8 + g;
+                    if (tk < p.m)
+                        b = p.x_smem ? *reinterpret_cast<const uint4 *>(s_x + tk * p.xs_stride + (cur.c + i) * 64 + t * 16)
+                                     : *reinterpret_cast<const uint4 *>(p.x + static_cast<size_t>(tk) * p.ldx + (cur.c + i) * 32 + t * 8);
 #pragma unroll
                     for (int a = 0; a < NA; ++a) {
-                        wl[a][i] = __ldcs(reinterpret_cast<const uint4 *>(w_lo + a * up + (c + i) * 32));
-                        wh[a][i] = __ldcs(reinterpret_cast<const uint4 *>(w_hi + a * up + (c + i) * 32));
+                        const uint32_t a0[4] = {wl[a][i].x, wh[a][i].x, wl[a][i].y, wh[a][i].y};
+                        const uint32_t a1[4] = {wl[a][i].z, wh[a][i].z, wl[a][i].w, wh[a][i].w};
+                        ptx::mma_bf16(acc[a][j], a0, b.x, b.y);
+                        ptx::mma_bf16(acc[a][j], a1, b.z, b.w);
                     }
                 }
+            }
+        const int tile = cur.tile, k0 = cur.k0, k1 = cur.k1;
+        cur = nxt;
 #pragma unroll
-            for (int i = 0; i < kFewUnroll; ++i)
-                if (c + i < c1) {
+        for (int w = 0; w < NA; ++w)
 #pragma unroll
-                    for (int j = 0; j < NTL; ++j) {
-                        uint4 b = make_uint4(0u, 0u, 0u, 0u);
-                        const int tk = j * 8 + g;
-                        if (tk < p.m)
-                            b = p.x_smem ? *reinterpret_cast<const uint4 *>(s_x + tk * p.xs_stride + (c + i) * 64 + t * 16)
-                                         : *reinterpret_cast<const uint4 *>(p.x + static_cast<size_t>(tk) * p.ldx + (c + i) * 32 + t * 8);
-#pragma unroll
-                        for (int a = 0; a < NA; ++a) {
-                            const uint32_t a0[4] = {wl[a][i].x, wh[a][i].x, wl[a][i].y, wh[a][i].y};
-                            const uint32_t a1[4] = {wl[a][i].z, wh[a][i].z, wl[a][i].w, wh[a][i].w};
-                            ptx::mma_bf16(acc[a][j], a0, b.x, b.y);
-                            ptx::mma_bf16(acc[a][j], a1, b.z, b.w);
-                        }
-                    }
-                }
-        }
+            for (int i = 0; i < U; ++i) {
+                wl[w][i] = nl[w][i];
+                wh[w][i] = nh[w][i];
+            }
+        if (!part_done) continue;
         // the sixteen K ranges meet: [warp][a][token][row], then one thread per output
         float *part = s_part + (buf * kFewWarps + warp) * kPart;
 #pragma unroll
@@ -200,18 +259,53 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
                 o[(2 * t + 1) * 16 + g] = acc[a][j][1];
                 o[(2 * t) * 16 + g + 8] = acc[a][j][2];
                 o[(2 * t + 1) * 16 + g + 8] = acc[a][j][3];
+                acc[a][j][0] = acc[a][j][1] = acc[a][j][2] = acc[a][j][3] = 0.0f;
             }
-        __syncthreads();  // the other buffer's readers passed this point one tile ago
-        for (int o = tid; o < NTL * 128; o += kFewThreads) {
-            const int tk = o >> 4, r = tile * 16 + (o & 15);
-            if (tk >= p.m || r >= p.out_rows) continue;
-            float v[NA];
+        buf ^= 1;         // the next part's sums go to the other buffer
+        __syncthreads();  // ... whose readers passed this point one part ago
+        const bool whole = k0 == 0 && k1 == p.chunks;
+        static_assert(NTL * 128 <= kFewThreads, "one thread per (token, row)");
+        const int o = tid, tk = o >> 4, r = tile * 16 + (o & 15);
+        const bool mine = o < NTL * 128 && tk < p.m && r < p.out_rows;
+        float v[NA];
+        if (mine) {
 #pragma unroll
             for (int a = 0; a < NA; ++a) {
                 v[a] = 0.0f;
 #pragma unroll
-                for (int w = 0; w < kFewWarps; ++w) v[a] += s_part[(buf * kFewWarps + w) * kPart + a * NTL * 128 + o];
+                for (int w = 0; w < kFewWarps; ++w) v[a] += s_part[((buf ^ 1) * kFewWarps + w) * kPart + a * NTL * 128 + o];
             }
+        }
+        if (!whole) {
+            // a tile shared with neighbouring CTAs: a CTA's first tile has slot 2c, its last one slot 2c + 1
+            auto slot = [&](int c) { return p.parts + static_cast<size_t>(2 * c + (c * p.per / p.chunks == tile ? 0 : 1)) * kFewPart; };
+            float *own = slot(blockIdx.x);
+            if (mine) {
+#pragma unroll
+                for (int a = 0; a < NA; ++a) __stcg(own + a * NTL * 128 + o, v[a]);
+            }
+            __threadfence();
+            __syncthreads();
+            const int first = tile * p.chunks / p.per, last = ((tile + 1) * p.chunks - 1) / p.per;
+            if (tid == 0) {
+                const int before = atomicAdd(p.counters + tile, 1);
+                s_last = before == last - first;
+                if (s_last) p.counters[tile] = 0;
+            }
+            __syncthreads();
+            if (!s_last) continue;
+            __threadfence();
+            if (mine) {
+#pragma unroll
+                for (int a = 0; a < NA; ++a) v[a] = 0.0f;
+                for (int c = first; c <= last; ++c) {
+                    const float *q = slot(c);
+#pragma unroll
+                    for (int a = 0; a < NA; ++a) v[a] += __ldcg(q + a * NTL * 128 + o);
+                }
+            }
+        }
+        if (mine) {
             const float val = DUAL ? dense::gelu_tanh<false>(v[0]) * v[NA - 1] : v[0];
             dense::row_store<uint16_t>(p.epi, dense::row_plan<uint16_t>(p.epi, r, pos0), tk, val);
         }
@@ -226,6 +320,7 @@ constexpr int kGStageBytes = 48 * 1024;         // one weight box + 256 tokens, 
 constexpr int kGBars = kGStages * kGStageBytes;
 constexpr int kGMisc = kGBars + 32 * 8;
 constexpr int kGMaxExperts = 1024;
+constexpr int kGSplitCtas = 128;                // CTAs of a launch that splits K over clusters
 constexpr int kGSmem = kGMisc + 64 + 1024;
 constexpr int kGThreads = 6 * 32;               // warps 0-3 epilogue, 4 TMA, 5 MMA
 
@@ -237,7 +332,22 @@ struct GemmParams {
     int experts, group_rows;
     const int *offs;
     int *err_word;
+    int ksplit, kb_part;    // CTAs per tile (the cluster's size), K blocks each
 };
+
+__device__ __forceinline__ void cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release;\nbarrier.cluster.wait.acquire;" ::: "memory");
+}
+__device__ __forceinline__ uint32_t peer_smem(uint32_t addr, int rank) {
+    uint32_t d;
+    asm("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(d) : "r"(addr), "r"(rank));
+    return d;
+}
+__device__ __forceinline__ float ld_peer(uint32_t addr) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+    return v;
+}
 
 __device__ __forceinline__ void umma4(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate_first) {
     asm volatile(
@@ -286,7 +396,7 @@ struct TileWalk {
     }
 };
 
-template <bool DUAL>
+template <bool DUAL, bool SPLIT>
 __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_constant__ GemmParams p) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ int s_end[kGMaxExperts];
@@ -334,23 +444,28 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
     ptx::pdl_trigger();
     bool ok = true;
     TileWalk walk(p, s_end);
+    // this CTA's tiles and K blocks; SPLIT: one tile per cluster, a part of its K per CTA
+    const int rank = SPLIT ? static_cast<int>(blockIdx.x) % p.ksplit : 0;
+    const int first = SPLIT ? static_cast<int>(blockIdx.x) / p.ksplit : static_cast<int>(blockIdx.x);
+    const int step = SPLIT ? tiles : static_cast<int>(gridDim.x);
+    const int kb0 = SPLIT ? rank * p.kb_part : 0;
+    const int kbn = SPLIT ? min(p.kb_part, p.k_blocks - kb0) : p.k_blocks;
 
     if (warp == 4) {
         // ================= TMA producer =================
         if (lane == 0) {
-            const int first = static_cast<int>(blockIdx.x), step = static_cast<int>(gridDim.x);
             const int my_tiles = tiles > first ? (tiles - first + step - 1) / step : 0;
-            const int total = my_tiles * p.k_blocks;
+            const int total = my_tiles * kbn;
             const uint32_t stage_tx = static_cast<uint32_t>(NA * kGWBytes + p.nt * 128);
             int row0, wrow = 0, tok0 = 0, ntok, s = 0, round = 0, kb = 0, tile = first;
             // Without experts the weights' first ring is on its way before the kernel in front is known to be complete.
             const int pre = p.experts ? 0 : (total < kGStages ? total : kGStages);
             for (int it = 0; it < pre; ++it) {
-                walk.get(first + (it / p.k_blocks) * step, row0, wrow, tok0, ntok);
+                walk.get(first + (it / kbn) * step, row0, wrow, tok0, ntok);
                 ptx::mbar_arrive_expect_tx(bar(kFull + it), stage_tx);
 #pragma unroll
                 for (int a = 0; a < NA; ++a)
-                    ptx::tma_load_2d(base + it * kGStageBytes + a * kGWBytes, &p.w, bar(kFull + it), (it % p.k_blocks) * 128, wrow + a * p.up_row);
+                    ptx::tma_load_2d(base + it * kGStageBytes + a * kGWBytes, &p.w, bar(kFull + it), (kb0 + it % kbn) * 128, wrow + a * p.up_row);
             }
             if (!p.experts) ptx::pdl_wait();
             for (int it = 0; it < total; ++it) {
@@ -363,14 +478,14 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
                     }
                     ptx::mbar_arrive_expect_tx(bar(kFull + s), stage_tx);
 #pragma unroll
-                    for (int a = 0; a < NA; ++a) ptx::tma_load_2d(st + a * kGWBytes, &p.w, bar(kFull + s), kb * 128, wrow + a * p.up_row);
+                    for (int a = 0; a < NA; ++a) ptx::tma_load_2d(st + a * kGWBytes, &p.w, bar(kFull + s), (kb0 + kb) * 128, wrow + a * p.up_row);
                 }
-                ptx::tma_load_2d(st + kXOff, &p.x, bar(kFull + s), kb * 128, tok0);
+                ptx::tma_load_2d(st + kXOff, &p.x, bar(kFull + s), (kb0 + kb) * 128, tok0);
                 if (++s == kGStages) {
                     s = 0;
                     ++round;
                 }
-                if (++kb == p.k_blocks) {
+                if (++kb == kbn) {
                     kb = 0;
                     tile += step;
                 }
@@ -382,7 +497,7 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
             const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(p.nt >> 3) << 17) | ((kGRows >> 4) << 24);
             const uint64_t adesc0 = smem_desc_sw128(base), bdesc0 = smem_desc_sw128(base + kXOff);
             int s = 0, phase = 0, tcount = 0;
-            for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++tcount) {
+            for (int tile = first; tile < tiles && ok; tile += step, ++tcount) {
                 const int a = tcount & 1, around = tcount >> 1;
                 if (around > 0 && !wait_bar(bar(kAccEmpty + a), (around - 1) & 1, s_abort)) {
                     ok = false;
@@ -390,7 +505,7 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
                 }
                 tc_fence_after();
                 const uint32_t d_tmem = tmem_base + a * 256;
-                for (int kb = 0; kb < p.k_blocks; ++kb) {
+                for (int kb = 0; kb < kbn; ++kb) {
                     if (!wait_bar(bar(kFull + s), phase, s_abort)) {
                         ok = false;
                         break;
@@ -416,7 +531,7 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
         int pos0 = 0;
         const bool fits = dense::rows_fit(p.epi, p.m, pos0);
         int tcount = 0;
-        for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++tcount) {
+        for (int tile = first; tile < tiles && ok; tile += step, ++tcount) {
             const int a = tcount & 1, around = tcount >> 1;
             int row0, wrow, tok0, ntok;
             walk.get(tile, row0, wrow, tok0, ntok);
@@ -425,6 +540,24 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
                 break;
             }
             tc_fence_after();
+            if (SPLIT) {
+                // this part's sums to shared memory, [accumulator][token][row] (the ring is free: every MMA has retired)
+                const uint32_t acc = tmem_base + (static_cast<uint32_t>(warp * 32) << 16);
+                float *mine = reinterpret_cast<float *>(sm) + warp * 32 + lane;
+#pragma unroll 1
+                for (int w2 = 0; w2 < NA; ++w2)
+#pragma unroll 1
+                    for (int c = 0; c * 32 < ntok; ++c) {
+                        uint32_t v[32];
+                        tmem_ld32(acc + w2 * kAccCols + c * 32, v);
+                        tmem_ld_wait();
+#pragma unroll
+                        for (int i = 0; i < 32; ++i)
+                            if (c * 32 + i < p.nt) mine[(w2 * p.nt + c * 32 + i) * kGRows] = __uint_as_float(v[i]);
+                    }
+                tc_fence_before();
+                break;
+            }
             const int row = row0 + warp * 32 + lane;
             dense::RowPlan plan;
             if (row < p.out_rows && fits) plan = dense::row_plan<uint16_t>(p.epi, row, pos0);
@@ -452,6 +585,31 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
             __syncwarp();
             if (lane == 0) ptx::mbar_arrive(bar(kAccEmpty + a));
         }
+    }
+    if (SPLIT) {
+        cluster_sync();  // every part's sums are in its CTA's shared memory
+        if (warp < 4) {
+            int pos0 = 0, row0, wrow, tok0, ntok;
+            const bool fits = dense::rows_fit(p.epi, p.m, pos0);
+            walk.get(first, row0, wrow, tok0, ntok);
+            const int row = row0 + warp * 32 + lane;
+            const int per = (ntok + p.ksplit - 1) / p.ksplit, t0 = rank * per, t1 = min(ntok, t0 + per);  // this CTA's tokens
+            if (row < p.out_rows && fits) {
+                const dense::RowPlan plan = dense::row_plan<uint16_t>(p.epi, row, pos0);
+                for (int t = t0; t < t1; ++t) {
+                    float v[NA];
+#pragma unroll
+                    for (int a = 0; a < NA; ++a) v[a] = 0.0f;
+                    for (int r = 0; r < p.ksplit; ++r) {
+                        const uint32_t peer = peer_smem(base + static_cast<uint32_t>((t * kGRows + warp * 32 + lane) * 4), r);
+#pragma unroll
+                        for (int a = 0; a < NA; ++a) v[a] += ld_peer(peer + static_cast<uint32_t>(a * p.nt * kGRows * 4));
+                    }
+                    dense::row_store<uint16_t>(p.epi, plan, tok0 + t, DUAL ? dense::gelu_tanh<false>(v[0]) * v[NA - 1] : v[0]);
+                }
+            }
+        }
+        cluster_sync();  // nobody leaves while its sums are being read
     }
     if (!ok && lane == 0) atomicExch(p.err_word, 5);
     tc_fence_before();
@@ -560,7 +718,21 @@ int launch_few(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
     p.x_smem = c.pre.mode != kPreNone || c.m * p.xs_stride <= kFewXSmem;
     const int ntl = c.m > 8 ? 2 : 1;
     const size_t smem = static_cast<size_t>(few_smem_bytes(p, ntl, c.gated));
-    const int grid = p.tiles < ctx->sm_count ? p.tiles : ctx->sm_count;
+    // Whole tiles, or equal runs of the (tile, K) stream when the idle SMs of the last round would cost more than the
+    // partial sums' trip through L2 (about 1.5 us; an SM streams about 40 bytes a nanosecond).
+    int grid = ctx->sm_count;
+    const int rounds = (p.tiles + grid - 1) / grid;
+    const double tile_us = static_cast<double>(p.chunks) * 1024.0 * (c.gated ? 2 : 1) / 40e3;
+    const double idle_us = (rounds - static_cast<double>(p.tiles) / grid) * tile_us;
+    if (idle_us > 1.5 && p.tiles <= kFewMaxTiles && grid <= kFewMaxCtas && ctx->few_parts) {
+        p.per = (p.tiles * p.chunks + grid - 1) / grid;
+        p.parts = static_cast<float *>(ctx->few_parts);
+        p.counters = reinterpret_cast<int *>(p.parts + static_cast<size_t>(2 * kFewMaxCtas) * kFewPart);
+        grid = (p.tiles * p.chunks + p.per - 1) / p.per;
+    } else {
+        p.per = rounds * p.chunks;
+        grid = (p.tiles + rounds - 1) / rounds;
+    }
     void (*k)(FewParams) = ntl == 1 ? (c.gated ? dense_few_kernel<1, true> : dense_few_kernel<1, false>)
                                     : (c.gated ? dense_few_kernel<2, true> : dense_few_kernel<2, false>);
     LBK_CUDA(launch_chained(k, dim3(static_cast<unsigned>(grid)), dim3(kFewThreads), smem, st, p));
@@ -612,9 +784,39 @@ int launch_gemm_tc(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
     p.err_word = ctx->err_word;
     LBK_TRY(encode_bytes_map(&p.w, c.w.w, c.w.pitch * 2, c.w.rows, c.w.pitch * 2, 128, kGRows));
     LBK_TRY(encode_bytes_map(&p.x, c.x, c.w.pitch * 2, c.m, static_cast<size_t>(c.ldx) * 2, 128, p.nt));
-    const int grid = !c.experts && p.tiles < ctx->sm_count ? p.tiles : ctx->sm_count;
-    LBK_CUDA(launch_chained(c.gated ? dense_gemm_kernel<true> : dense_gemm_kernel<false>, dim3(static_cast<unsigned>(grid)), dim3(kGThreads),
-                            static_cast<size_t>(kGSmem), st, p));
+    // K split over a cluster: at most kGSplitCtas CTAs in all (clusters live inside a GPC, so not every SM can be part
+    // of one), at least four K blocks each
+    p.ksplit = 1;
+    p.kb_part = p.k_blocks;
+    if (!c.experts)
+        for (int s = 8; s >= 2; s >>= 1) {
+            const int part = (p.k_blocks + s - 1) / s;
+            if (p.tiles * s <= kGSplitCtas && part >= 4 && part * (s - 1) < p.k_blocks && p.nt * (c.gated ? 2 : 1) * kGRows * 4 <= kGBars) {
+                p.ksplit = s;
+                p.kb_part = part;
+                break;
+            }
+        }
+    if (p.ksplit > 1) {
+        cudaLaunchConfig_t cfg{};
+        cfg.gridDim = dim3(static_cast<unsigned>(p.tiles * p.ksplit));
+        cfg.blockDim = dim3(kGThreads);
+        cfg.dynamicSmemBytes = kGSmem;
+        cfg.stream = st;
+        cudaLaunchAttribute attr[2]{};
+        attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[0].val.programmaticStreamSerializationAllowed = 1;
+        attr[1].id = cudaLaunchAttributeClusterDimension;
+        attr[1].val.clusterDim.x = static_cast<unsigned>(p.ksplit);
+        attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+        cfg.attrs = attr;
+        cfg.numAttrs = 2;
+        LBK_CUDA(cudaLaunchKernelEx(&cfg, c.gated ? dense_gemm_kernel<true, true> : dense_gemm_kernel<false, true>, p));
+    } else {
+        const int grid = !c.experts && p.tiles < ctx->sm_count ? p.tiles : ctx->sm_count;
+        LBK_CUDA(launch_chained(c.gated ? dense_gemm_kernel<true, false> : dense_gemm_kernel<false, false>, dim3(static_cast<unsigned>(grid)), dim3(kGThreads),
+                                static_cast<size_t>(kGSmem), st, p));
+    }
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;
     return LBK_OK;
@@ -644,14 +846,19 @@ int launch_f32(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
 }
 
 int dense_init(Ctx *ctx) {
+    constexpr size_t parts = static_cast<size_t>(2 * kFewMaxCtas) * kFewPart * sizeof(float) + kFewMaxTiles * sizeof(int);
+    LBK_CUDA(cudaMalloc(&ctx->few_parts, parts));
+    LBK_CUDA(cudaMemset(ctx->few_parts, 0, parts));
     const int few_max = 2 * kFewWarps * 2 * 2 * 128 * 4 + static_cast<int>(kFewXSmem);
     LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
     LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
     LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
     LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
     if (static_cast<size_t>(kGSmem) > ctx->smem_optin) return fail(LBK_ERR_UNSUPPORTED, "dense GEMM kernel needs %d B of shared memory", kGSmem);
-    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
-    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
+    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
+    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
+    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
+    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
     return LBK_OK;
 }
 const InitHook kInitDense(dense_init);

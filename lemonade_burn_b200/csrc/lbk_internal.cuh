@@ -52,6 +52,7 @@ struct Ctx {
     cudaStream_t own_stream = nullptr;  // used by the host-pointer entry points
     void *bf16_x = nullptr;             // allocated once at init: the bf16 head's activations as two bf16 terms (one pass of 64 token rows)
     void *small_scratch = nullptr;      // kSmallScratchBytes, allocated once at init (reductions)
+    void *few_parts = nullptr;          // allocated once at init: partial tiles and counters of the few-token bf16 projections
     int32_t *gemm_acc = nullptr;        // kGemmAccBytes, allocated once at init: int32 sums of a prefill GEMM split along K
     int gemv_rows = 0;                  // lbk_set_gemv_rows: 0 = measured rule, n = fused kernel up to n token rows
 };

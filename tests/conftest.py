@@ -32,7 +32,7 @@ def pytest_collection_modifyitems(config, items):
 
 @pytest.fixture(scope="session")
 def oracle():
-    """The CPU oracle (checker only)."""
+    """The CPU oracle (test infrastructure only)."""
     from oracle import oracle as o
     o.build()
     return o

@@ -26,8 +26,8 @@ def configs():
             a(20, 2, 64, 72, 150, 70, 0.4, d(448)),
             a(8, 1, 128, 128, 64, 1, 0.25, m(24, 6, 160, 200)),
             a(16, 8, 96, 64, 131, 129, 0.3, d(200))], eps=1e-5),
-        # one head, one key/value head, one expert: values other models make larger
-        "ones": p.make_config(65, 64, [a(1, 1, 64, 64, 8, 1, 1.0, m(1, 1, 64, 64)), a(1, 1, 16, 32, 1000, 0, 1.0, d(16))], eps=1e-6),
+        # one head, one key/value head, one expert (values other models make larger), and a width of no whole unit
+        "ones": p.make_config(65, 66, [a(1, 1, 64, 64, 8, 1, 1.0, m(1, 1, 64, 64)), a(1, 1, 16, 32, 1000, 0, 1.0, d(18))], eps=1e-6),
     }
 
 
