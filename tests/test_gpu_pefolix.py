@@ -28,6 +28,8 @@ def configs():
             a(16, 8, 96, 64, 131, 129, 0.3, d(200))], eps=1e-5),
         # one head, one key/value head, one expert (values other models make larger), and a width of no whole unit
         "ones": p.make_config(65, 66, [a(1, 1, 64, 64, 8, 1, 1.0, m(1, 1, 64, 64)), a(1, 1, 16, 32, 1000, 0, 1.0, d(18))], eps=1e-6),
+        # more experts than the usual routing kernel holds
+        "many": p.make_config(90, 48, [a(2, 1, 32, 32, 50, 2, 0.5, m(300, 3, 12, 20))], eps=1e-5),
     }
 
 
@@ -80,7 +82,7 @@ def logits(nets, name, toks):
 
 
 @pytest.mark.parametrize("dtype", list(TOL))
-@pytest.mark.parametrize("name", ["mixed", "wide", "ones"])
+@pytest.mark.parametrize("name", ["mixed", "wide", "ones", "many"])
 def test_whole_prompts(nets, name, dtype):
     cfg, _, models = nets[name]
     net = models[dtype]
@@ -93,7 +95,7 @@ def test_whole_prompts(nets, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", list(TOL))
-@pytest.mark.parametrize("name", ["mixed", "wide", "ones"])
+@pytest.mark.parametrize("name", ["mixed", "wide", "ones", "many"])
 def test_token_by_token_and_long_decoding(nets, name, dtype):
     """The recorded decode step from position 0 to 260 (past every window, with kept tokens), and the same tokens as a
     prompt of 200 followed by single ones."""
