@@ -2,7 +2,7 @@
 // epilogue (lbk_dense_dev.cuh: f32 rows, activated rows in the compute type, or [q; k; v] rows of which k and v
 // go straight into the cache):
 //
-//   dense_few_kernel   up to 16 tokens (decode, short portions). Bound: HBM, the weights once. 16 weight rows
+//   dense_few_kernel   up to 8 tokens (decode, short portions). Bound: HBM, the weights once. 16 weight rows
 //                      are the M side of mma.sync m16n8k16, the tokens its N side; a lane's 16-byte weight load
 //                      is two MMAs' operands as it is (the contraction index may be permuted as long as both
 //                      operands are permuted alike), so weights go global -> registers -> tensor core without
@@ -15,7 +15,10 @@
 //                      by TMA (SWIZZLE_128B, 64 columns a stage), two accumulators in tensor memory so that the
 //                      epilogue of one tile runs under the MMAs of the next, one persistent CTA per SM. A gated
 //                      projection keeps gate and up accumulators of the same 128 rows side by side, so the
-//                      product is taken where both sit in one thread's registers. Few tiles and a long K (a short
+//                      product is taken where both sit in one thread's registers. Large calls are bound by the
+//                      operands' way into the SMs (48 KB per 128 x 256 x 64 block): they take the wide form, two
+//                      weight boxes x up to 256 tokens (64 KB for twice the block), whose accumulators fill tensor
+//                      memory, so its epilogue is not hidden; choose_tile weighs the two. Few tiles and a long K (a short
 //                      portion of a prompt) are cut along K over a cluster of 2 to 8 CTAs, whose accumulators meet
 //                      in shared memory: every CTA reads its share of the tokens from all of them, in rank order.
 //                      With experts the tokens
@@ -34,10 +37,11 @@ using namespace tc;
 
 // ---- few tokens ---------------------------------------------------------------------------------
 constexpr int kFewThreads = 512, kFewWarps = 16;
+constexpr int kFewTokens = 8;               // up to here; 9 to 16 tokens run faster on dense_gemm_kernel (14336 -> 4096: 26 against 38 us)
 constexpr int kFewPreMax = 2;               // tokens whose norms run in the prologue
 constexpr size_t kFewXSmem = 96 * 1024;     // activations in shared memory up to this, else read through L1
 
-constexpr int kFewPart = 2 * 2 * 128;       // floats of a partial tile: gate and up, 16 tokens, 16 rows
+constexpr int kFewPart = 2 * 128;           // floats of a partial tile: gate and up, 8 tokens, 16 rows
 constexpr int kFewMaxTiles = 1 << 14, kFewMaxCtas = 512;
 constexpr int kFewPrefetch = 2;             // 128-byte lines a thread asks L2 for ahead of the kernel in front
 
@@ -123,12 +127,12 @@ __device__ __forceinline__ void few_norm_row(const FewParams &p, int t, bool wri
     }
 }
 
-template <int NTL, bool DUAL>
+template <bool DUAL>
 __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_constant__ FewParams p) {
     extern __shared__ __align__(16) uint8_t few_smem[];
     __shared__ float s_red[32];
     constexpr int NA = DUAL ? 2 : 1;
-    constexpr int kPart = NA * NTL * 128;   // floats a warp contributes per tile
+    constexpr int kPart = NA * 128;         // floats a warp contributes per tile
     float *s_part = reinterpret_cast<float *>(few_smem);               // [2][16 warps][kPart]
     uint8_t *s_x = few_smem + 2 * kFewWarps * kPart * sizeof(float);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
@@ -196,11 +200,10 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
                 }
             }
     };
-    float acc[NA][NTL][4];
+    float acc[NA][4];
 #pragma unroll
     for (int a = 0; a < NA; ++a)
-#pragma unroll
-        for (int j = 0; j < NTL; ++j) acc[a][j][0] = acc[a][j][1] = acc[a][j][2] = acc[a][j][3] = 0.0f;
+        acc[a][0] = acc[a][1] = acc[a][2] = acc[a][3] = 0.0f;
     int buf = 0;
     Step cur, nxt;
     bool more = at < s_end;
@@ -222,20 +225,16 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
 #pragma unroll
         for (int i = 0; i < U; ++i)
             if (cur.c + i < cur.c1) {
+                uint4 b = make_uint4(0u, 0u, 0u, 0u);
+                if (g < p.m)
+                    b = p.x_smem ? *reinterpret_cast<const uint4 *>(s_x + g * p.xs_stride + (cur.c + i) * 64 + t * 16)
+                                 : *reinterpret_cast<const uint4 *>(p.x + static_cast<size_t>(g) * p.ldx + (cur.c + i) * 32 + t * 8);
 #pragma unroll
-                for (int j = 0; j < NTL; ++j) {
-                    uint4 b = make_uint4(0u, 0u, 0u, 0u);
-                    const int tk = j * 8 + g;
-                    if (tk < p.m)
-                        b = p.x_smem ? *reinterpret_cast<const uint4 *>(s_x + tk * p.xs_stride + (cur.c + i) * 64 + t * 16)
-                                     : *reinterpret_cast<const uint4 *>(p.x + static_cast<size_t>(tk) * p.ldx + (cur.c + i) * 32 + t * 8);
-#pragma unroll
-                    for (int a = 0; a < NA; ++a) {
-                        const uint32_t a0[4] = {wl[a][i].x, wh[a][i].x, wl[a][i].y, wh[a][i].y};
-                        const uint32_t a1[4] = {wl[a][i].z, wh[a][i].z, wl[a][i].w, wh[a][i].w};
-                        ptx::mma_bf16(acc[a][j], a0, b.x, b.y);
-                        ptx::mma_bf16(acc[a][j], a1, b.z, b.w);
-                    }
+                for (int a = 0; a < NA; ++a) {
+                    const uint32_t a0[4] = {wl[a][i].x, wh[a][i].x, wl[a][i].y, wh[a][i].y};
+                    const uint32_t a1[4] = {wl[a][i].z, wh[a][i].z, wl[a][i].w, wh[a][i].w};
+                    ptx::mma_bf16(acc[a], a0, b.x, b.y);
+                    ptx::mma_bf16(acc[a], a1, b.z, b.w);
                 }
             }
         const int tile = cur.tile, k0 = cur.k0, k1 = cur.k1;
@@ -251,29 +250,27 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
         // the sixteen K ranges meet: [warp][a][token][row], then one thread per output
         float *part = s_part + (buf * kFewWarps + warp) * kPart;
 #pragma unroll
-        for (int a = 0; a < NA; ++a)
-#pragma unroll
-            for (int j = 0; j < NTL; ++j) {
-                float *o = part + (a * NTL + j) * 128;
-                o[(2 * t) * 16 + g] = acc[a][j][0];
-                o[(2 * t + 1) * 16 + g] = acc[a][j][1];
-                o[(2 * t) * 16 + g + 8] = acc[a][j][2];
-                o[(2 * t + 1) * 16 + g + 8] = acc[a][j][3];
-                acc[a][j][0] = acc[a][j][1] = acc[a][j][2] = acc[a][j][3] = 0.0f;
-            }
+        for (int a = 0; a < NA; ++a) {
+            float *o = part + a * 128;
+            o[(2 * t) * 16 + g] = acc[a][0];
+            o[(2 * t + 1) * 16 + g] = acc[a][1];
+            o[(2 * t) * 16 + g + 8] = acc[a][2];
+            o[(2 * t + 1) * 16 + g + 8] = acc[a][3];
+            acc[a][0] = acc[a][1] = acc[a][2] = acc[a][3] = 0.0f;
+        }
         buf ^= 1;         // the next part's sums go to the other buffer
         __syncthreads();  // ... whose readers passed this point one part ago
         const bool whole = k0 == 0 && k1 == p.chunks;
-        static_assert(NTL * 128 <= kFewThreads, "one thread per (token, row)");
+        static_assert(kFewTokens == 8, "one MMA tile of tokens; 128 (token, row) pairs, a thread each");
         const int o = tid, tk = o >> 4, r = tile * 16 + (o & 15);
-        const bool mine = o < NTL * 128 && tk < p.m && r < p.out_rows;
+        const bool mine = o < 128 && tk < p.m && r < p.out_rows;
         float v[NA];
         if (mine) {
 #pragma unroll
             for (int a = 0; a < NA; ++a) {
                 v[a] = 0.0f;
 #pragma unroll
-                for (int w = 0; w < kFewWarps; ++w) v[a] += s_part[((buf ^ 1) * kFewWarps + w) * kPart + a * NTL * 128 + o];
+                for (int w = 0; w < kFewWarps; ++w) v[a] += s_part[((buf ^ 1) * kFewWarps + w) * kPart + a * 128 + o];
             }
         }
         if (!whole) {
@@ -282,7 +279,7 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
             float *own = slot(blockIdx.x);
             if (mine) {
 #pragma unroll
-                for (int a = 0; a < NA; ++a) __stcg(own + a * NTL * 128 + o, v[a]);
+                for (int a = 0; a < NA; ++a) __stcg(own + a * 128 + o, v[a]);
             }
             __threadfence();
             __syncthreads();
@@ -301,7 +298,7 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
                 for (int c = first; c <= last; ++c) {
                     const float *q = slot(c);
 #pragma unroll
-                    for (int a = 0; a < NA; ++a) v[a] += __ldcg(q + a * NTL * 128 + o);
+                    for (int a = 0; a < NA; ++a) v[a] += __ldcg(q + a * 128 + o);
                 }
             }
         }
@@ -313,22 +310,23 @@ __global__ void __launch_bounds__(kFewThreads, 1) dense_few_kernel(const __grid_
 }
 
 // ---- many tokens: tcgen05 -------------------------------------------------------------------------
-constexpr int kGRows = 128;                     // weight rows per tile (MMA M, TMEM lanes)
-constexpr int kGStages = 4;
+constexpr int kGRows = 128;                     // weight rows per box (MMA M, TMEM lanes)
 constexpr int kGWBytes = kGRows * 128;          // 16 KB: 128 rows x 64 columns
-constexpr int kGStageBytes = 48 * 1024;         // one weight box + 256 tokens, or two weight boxes + 128 tokens
-constexpr int kGBars = kGStages * kGStageBytes;
+constexpr int kGRing = 192 * 1024;              // four stages of 48 KB (one weight box + 256 tokens, or two + 128), wide: three of 64 KB
+constexpr int kGBars = kGRing;
 constexpr int kGMisc = kGBars + 32 * 8;
 constexpr int kGMaxExperts = 1024;
 constexpr int kGSplitCtas = 128;                // CTAs of a launch that splits K over clusters
 constexpr int kGSmem = kGMisc + 64 + 1024;
-constexpr int kGThreads = 6 * 32;               // warps 0-3 epilogue, 4 TMA, 5 MMA
+constexpr int kGEpiWarps = 8, kGTmaWarp = 8, kGMmaWarp = 9;
+constexpr int kGThreads = 10 * 32;
+constexpr int kGated = 1, kWide = 2;            // KIND bits
 
 struct GemmParams {
     CUtensorMap w;      // bytes [stacked rows][pitch * 2], box [128][128]
     CUtensorMap x;      // bytes [tokens][ldx * 2], box [nt][128]
     DenseEpi epi;
-    int out_rows, up_row, k_blocks, m, nt, row_tiles, token_tiles, tiles;
+    int out_rows, box2_row, tile_rows, k_blocks, m, nt, row_tiles, token_tiles, tiles;  // box2_row: rows from the first weight box to the second
     int experts, group_rows;
     const int *offs;
     int *err_word;
@@ -380,7 +378,7 @@ struct TileWalk {
     __device__ __forceinline__ void get(int tile, int &row0, int &wrow, int &tok0, int &ntok) {
         if (!p.experts) {
             const int rt = tile / p.token_tiles, tt = tile - rt * p.token_tiles;
-            row0 = wrow = rt * kGRows;
+            row0 = wrow = rt * p.tile_rows;
             tok0 = tt * p.nt;
             ntok = min(p.nt, p.m - tok0);
             return;
@@ -389,20 +387,23 @@ struct TileWalk {
         const int first = e ? s_end[e - 1] : 0, local = tile - first;
         const int b = p.offs[e], cnt = p.offs[e + 1] - b, tts = (cnt + p.nt - 1) / p.nt;
         const int rt = local / tts, tt = local - rt * tts;
-        row0 = rt * kGRows;
+        row0 = rt * p.tile_rows;
         wrow = e * p.group_rows + row0;
         tok0 = b + tt * p.nt;
         ntok = min(p.nt, cnt - tt * p.nt);
     }
 };
 
-template <bool DUAL, bool SPLIT>
+template <int KIND, bool SPLIT>
 __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_constant__ GemmParams p) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ int s_end[kGMaxExperts];
-    constexpr int NA = DUAL ? 2 : 1;
+    constexpr bool GATED = (KIND & kGated) != 0, WIDE = (KIND & kWide) != 0;
+    constexpr int NA = KIND ? 2 : 1;            // weight boxes a stage
+    constexpr int kGStages = WIDE ? 3 : 4, kGStageBytes = kGRing / kGStages;
     constexpr int kXOff = NA * kGWBytes;
-    constexpr int kAccCols = DUAL ? 128 : 256;  // columns of one accumulator; two sets of NA of them fill tensor memory
+    constexpr int kAccCols = KIND == kGated ? 128 : 256;  // columns of one accumulator
+    constexpr int NB = WIDE ? 1 : 2;            // sets of NA accumulators: NB * NA * kAccCols = 512 columns
     const uint32_t raw = ptx::smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
     uint8_t *sm = smem_raw + (base - raw);
@@ -419,12 +420,12 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
         }
         for (int a = 0; a < 2; ++a) {
             ptx::mbar_init(bar(kAccFull + a), 1);
-            ptx::mbar_init(bar(kAccEmpty + a), 4);
+            ptx::mbar_init(bar(kAccEmpty + a), kGEpiWarps);
         }
         *s_abort = 0;
         ptx::fence_barrier_init();
     }
-    if (warp == 5) {
+    if (warp == kGMmaWarp) {
         tmem_alloc(base + kGMisc, 512);
         tmem_relinquish();
     }
@@ -451,7 +452,7 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
     const int kb0 = SPLIT ? rank * p.kb_part : 0;
     const int kbn = SPLIT ? min(p.kb_part, p.k_blocks - kb0) : p.k_blocks;
 
-    if (warp == 4) {
+    if (warp == kGTmaWarp) {
         // ================= TMA producer =================
         if (lane == 0) {
             const int my_tiles = tiles > first ? (tiles - first + step - 1) / step : 0;
@@ -465,7 +466,7 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
                 ptx::mbar_arrive_expect_tx(bar(kFull + it), stage_tx);
 #pragma unroll
                 for (int a = 0; a < NA; ++a)
-                    ptx::tma_load_2d(base + it * kGStageBytes + a * kGWBytes, &p.w, bar(kFull + it), (kb0 + it % kbn) * 128, wrow + a * p.up_row);
+                    ptx::tma_load_2d(base + it * kGStageBytes + a * kGWBytes, &p.w, bar(kFull + it), (kb0 + it % kbn) * 128, wrow + a * p.box2_row);
             }
             if (!p.experts) ptx::pdl_wait();
             for (int it = 0; it < total; ++it) {
@@ -478,7 +479,7 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
                     }
                     ptx::mbar_arrive_expect_tx(bar(kFull + s), stage_tx);
 #pragma unroll
-                    for (int a = 0; a < NA; ++a) ptx::tma_load_2d(st + a * kGWBytes, &p.w, bar(kFull + s), (kb0 + kb) * 128, wrow + a * p.up_row);
+                    for (int a = 0; a < NA; ++a) ptx::tma_load_2d(st + a * kGWBytes, &p.w, bar(kFull + s), (kb0 + kb) * 128, wrow + a * p.box2_row);
                 }
                 ptx::tma_load_2d(st + kXOff, &p.x, bar(kFull + s), (kb0 + kb) * 128, tok0);
                 if (++s == kGStages) {
@@ -491,14 +492,14 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
                 }
             }
         }
-    } else if (warp == 5) {
+    } else if (warp == kGMmaWarp) {
         // ================= MMA issuer (one thread) =================
         if (lane == 0) {
             const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(p.nt >> 3) << 17) | ((kGRows >> 4) << 24);
             const uint64_t adesc0 = smem_desc_sw128(base), bdesc0 = smem_desc_sw128(base + kXOff);
             int s = 0, phase = 0, tcount = 0;
             for (int tile = first; tile < tiles && ok; tile += step, ++tcount) {
-                const int a = tcount & 1, around = tcount >> 1;
+                const int a = tcount % NB, around = tcount / NB;
                 if (around > 0 && !wait_bar(bar(kAccEmpty + a), (around - 1) & 1, s_abort)) {
                     ok = false;
                     break;
@@ -526,13 +527,14 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
             }
         }
     } else {
-        // ================= epilogue (warps 0..3 = TMEM lane quadrants 0..3) =================
+        // ================= epilogue (warps w and w + 4: TMEM lane quadrant w & 3) =================
         if (!p.experts) ptx::pdl_wait();  // outputs may still be read by the kernel in front; the position is its
         int pos0 = 0;
         const bool fits = dense::rows_fit(p.epi, p.m, pos0);
+        const int quad = warp & 3, half = warp >> 2;  // half: one of two plain weight boxes, or every second 32 tokens
         int tcount = 0;
         for (int tile = first; tile < tiles && ok; tile += step, ++tcount) {
-            const int a = tcount & 1, around = tcount >> 1;
+            const int a = tcount % NB, around = tcount / NB;
             int row0, wrow, tok0, ntok;
             walk.get(tile, row0, wrow, tok0, ntok);
             if (!__all_sync(0xffffffffu, wait_bar(bar(kAccFull + a), around & 1, s_abort))) {
@@ -542,12 +544,12 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
             tc_fence_after();
             if (SPLIT) {
                 // this part's sums to shared memory, [accumulator][token][row] (the ring is free: every MMA has retired)
-                const uint32_t acc = tmem_base + (static_cast<uint32_t>(warp * 32) << 16);
-                float *mine = reinterpret_cast<float *>(sm) + warp * 32 + lane;
+                const uint32_t acc = tmem_base + (static_cast<uint32_t>(quad * 32) << 16);
+                float *mine = reinterpret_cast<float *>(sm) + quad * 32 + lane;
 #pragma unroll 1
                 for (int w2 = 0; w2 < NA; ++w2)
 #pragma unroll 1
-                    for (int c = 0; c * 32 < ntok; ++c) {
+                    for (int c = half; c * 32 < ntok; c += 2) {
                         uint32_t v[32];
                         tmem_ld32(acc + w2 * kAccCols + c * 32, v);
                         tmem_ld_wait();
@@ -558,15 +560,15 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
                 tc_fence_before();
                 break;
             }
-            const int row = row0 + warp * 32 + lane;
+            const int row = row0 + (KIND == kWide ? half * kGRows : 0) + quad * 32 + lane;
             dense::RowPlan plan;
             if (row < p.out_rows && fits) plan = dense::row_plan<uint16_t>(p.epi, row, pos0);
-            const uint32_t acc = tmem_base + (static_cast<uint32_t>(warp * 32) << 16) + a * 256;
+            const uint32_t acc = tmem_base + (static_cast<uint32_t>(quad * 32) << 16) + (KIND == kWide ? half * kAccCols : a * 256);
 #pragma unroll 1
-            for (int c = 0; c * 32 < ntok; ++c) {
+            for (int c = KIND == kWide ? 0 : half; c * 32 < ntok; c += KIND == kWide ? 1 : 2) {
                 uint32_t v[32];
                 tmem_ld32(acc + c * 32, v);
-                if (DUAL) {
+                if (GATED) {
                     uint32_t u[32];
                     tmem_ld32(acc + kAccCols + c * 32, u);
                     tmem_ld_wait();
@@ -588,24 +590,38 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
     }
     if (SPLIT) {
         cluster_sync();  // every part's sums are in its CTA's shared memory
-        if (warp < 4) {
+        if (warp < kGEpiWarps) {
             int pos0 = 0, row0, wrow, tok0, ntok;
             const bool fits = dense::rows_fit(p.epi, p.m, pos0);
             walk.get(first, row0, wrow, tok0, ntok);
-            const int row = row0 + warp * 32 + lane;
+            const int lane_row = (warp & 3) * 32 + lane, row = row0 + lane_row;
             const int per = (ntok + p.ksplit - 1) / p.ksplit, t0 = rank * per, t1 = min(ntok, t0 + per);  // this CTA's tokens
             if (row < p.out_rows && fits) {
                 const dense::RowPlan plan = dense::row_plan<uint16_t>(p.epi, row, pos0);
-                for (int t = t0; t < t1; ++t) {
-                    float v[NA];
+                constexpr int TU = 4;  // tokens at a time: their loads from the other SMs are in flight together
+                for (int t = t0 + (warp >> 2); t < t1; t += 2 * TU) {
+                    float v[TU][NA];
 #pragma unroll
-                    for (int a = 0; a < NA; ++a) v[a] = 0.0f;
+                    for (int i = 0; i < TU; ++i)
+#pragma unroll
+                        for (int a = 0; a < NA; ++a) v[i][a] = 0.0f;
                     for (int r = 0; r < p.ksplit; ++r) {
-                        const uint32_t peer = peer_smem(base + static_cast<uint32_t>((t * kGRows + warp * 32 + lane) * 4), r);
+                        const uint32_t peer = peer_smem(base + static_cast<uint32_t>(lane_row * 4), r);
+                        float w[TU][NA];
 #pragma unroll
-                        for (int a = 0; a < NA; ++a) v[a] += ld_peer(peer + static_cast<uint32_t>(a * p.nt * kGRows * 4));
+                        for (int i = 0; i < TU; ++i)
+#pragma unroll
+                            for (int a = 0; a < NA; ++a)
+                                w[i][a] = ld_peer(peer + static_cast<uint32_t>((a * p.nt + min(t + 2 * i, t1 - 1)) * kGRows * 4));
+#pragma unroll
+                        for (int i = 0; i < TU; ++i)
+#pragma unroll
+                            for (int a = 0; a < NA; ++a) v[i][a] += w[i][a];
                     }
-                    dense::row_store<uint16_t>(p.epi, plan, tok0 + t, DUAL ? dense::gelu_tanh<false>(v[0]) * v[NA - 1] : v[0]);
+#pragma unroll
+                    for (int i = 0; i < TU; ++i)
+                        if (t + 2 * i < t1)
+                            dense::row_store<uint16_t>(p.epi, plan, tok0 + t + 2 * i, GATED ? dense::gelu_tanh<false>(v[i][0]) * v[i][NA - 1] : v[i][0]);
                 }
             }
         }
@@ -614,7 +630,7 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
     if (!ok && lane == 0) atomicExch(p.err_word, 5);
     tc_fence_before();
     __syncthreads();
-    if (warp == 5) {
+    if (warp == kGMmaWarp) {
         tc_fence_after();
         tmem_dealloc(tmem_base, 512);
     }
@@ -696,8 +712,8 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const F32Params p) {
     }
 }
 
-int few_smem_bytes(const FewParams &p, int ntl, bool dual) {
-    return 2 * kFewWarps * (dual ? 2 : 1) * ntl * 128 * static_cast<int>(sizeof(float)) + (p.x_smem ? p.m * p.xs_stride : 0);
+int few_smem_bytes(const FewParams &p, bool dual) {
+    return 2 * kFewWarps * (dual ? 2 : 1) * 128 * static_cast<int>(sizeof(float)) + (p.x_smem ? p.m * p.xs_stride : 0);
 }
 
 int launch_few(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
@@ -716,8 +732,7 @@ int launch_few(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
     p.n = static_cast<int>(c.w.cols);
     p.xs_stride = static_cast<int>(c.w.pitch * 2 + 64);  // eight token rows start in different bank groups
     p.x_smem = c.pre.mode != kPreNone || c.m * p.xs_stride <= kFewXSmem;
-    const int ntl = c.m > 8 ? 2 : 1;
-    const size_t smem = static_cast<size_t>(few_smem_bytes(p, ntl, c.gated));
+    const size_t smem = static_cast<size_t>(few_smem_bytes(p, c.gated));
     // Whole tiles, or equal runs of the (tile, K) stream when the idle SMs of the last round would cost more than the
     // partial sums' trip through L2 (about 1.5 us; an SM streams about 40 bytes a nanosecond).
     int grid = ctx->sm_count;
@@ -733,27 +748,51 @@ int launch_few(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
         p.per = rounds * p.chunks;
         grid = (p.tiles + rounds - 1) / rounds;
     }
-    void (*k)(FewParams) = ntl == 1 ? (c.gated ? dense_few_kernel<1, true> : dense_few_kernel<1, false>)
-                                    : (c.gated ? dense_few_kernel<2, true> : dense_few_kernel<2, false>);
+    void (*k)(FewParams) = c.gated ? dense_few_kernel<true> : dense_few_kernel<false>;
     LBK_CUDA(launch_chained(k, dim3(static_cast<unsigned>(grid)), dim3(kFewThreads), smem, st, p));
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;
     return LBK_OK;
 }
 
-// Tokens per tile: the split of m that finishes first, counting whole rounds of tiles over the SMs (a tile of few
-// tokens costs as much as one of about 96: the weight side of the MMA then sets the pace).
-int choose_tokens(size_t m, size_t row_tiles, int limit, int sms) {
-    int best = limit;
+// CTAs a tile's K is cut over (a cluster), 1 when it is not worth it or the tiles are many: at most kGSplitCtas CTAs in
+// all (clusters live inside a GPC, so not every SM can be part of one), at least four K blocks each.
+int choose_ksplit(size_t tiles, int k_blocks, int boxes, int nt) {
+    for (int s = 8; s >= 2; s >>= 1) {
+        const int part = (k_blocks + s - 1) / s;
+        if (tiles * s <= static_cast<size_t>(kGSplitCtas) && part >= 4 && part * (s - 1) < k_blocks && nt * boxes * kGRows * 4 <= kGRing) return s;
+    }
+    return 1;
+}
+
+// Tile shape: the one that finishes first, counting whole rounds of tiles over the SMs. Cycles per 64 columns of K: the
+// MMAs' (two per token and weight box), or the operands' bytes at what an SM takes in beside 147 others (45 a cycle). The
+// wide form adds its epilogue, a split K the exchange of the sums.
+struct TileShape {
+    int nt = 16, ksplit = 1;
+    bool wide = false;
+};
+TileShape choose_tile(size_t m, size_t rows, int k_blocks, bool gated, int sms) {
+    TileShape best;
     double best_cost = 1e30;
-    for (int nt = 16; nt <= limit; nt += 16) {
-        const size_t tiles = (m + nt - 1) / nt * row_tiles;
-        const double cost = static_cast<double>((tiles + sms - 1) / sms) * ((nt < 96 ? 96 : nt) + 16);
-        if (cost <= best_cost) {
-            best_cost = cost;
-            best = nt;
+    for (int wide = 0; wide < 2; ++wide) {
+        const int boxes = gated || wide ? 2 : 1, limit = boxes == 2 && !wide ? 128 : 256;
+        const size_t tile_rows = wide && !gated ? 2 * kGRows : kGRows, row_tiles = (rows + tile_rows - 1) / tile_rows;
+        for (int nt = 16; nt <= limit; nt += 16) {
+            const size_t tiles = (m + nt - 1) / nt * row_tiles;
+            const int ksplit = wide ? 1 : choose_ksplit(tiles, k_blocks, boxes, nt);
+            const double mma = 2.0 * boxes * nt, bytes = (boxes * kGWBytes + nt * 128) / 45.0;
+            double cost = static_cast<double>((tiles + sms - 1) / sms) * (mma > bytes ? mma : bytes) * k_blocks;
+            if (ksplit > 1) cost = cost / ksplit + 3000.0 + 30.0 * boxes * nt;
+            if (wide) cost += static_cast<double>((tiles + sms - 1) / sms) * (gated ? 7000.0 : 3000.0);
+            if (cost <= best_cost) {
+                best_cost = cost;
+                best.nt = nt;
+                best.ksplit = ksplit;
+                best.wide = wide != 0;
+            }
+            if (static_cast<size_t>(nt) >= m) break;
         }
-        if (static_cast<size_t>(nt) >= m) break;
     }
     return best;
 }
@@ -763,10 +802,11 @@ int launch_gemm_tc(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
     GemmParams p{};
     p.epi = c.epi;
     p.out_rows = static_cast<int>(c.out_rows);
-    p.up_row = static_cast<int>(c.up_row);
     p.k_blocks = static_cast<int>(c.w.pitch / 64);
     p.m = static_cast<int>(c.m);
-    p.row_tiles = static_cast<int>((c.out_rows + kGRows - 1) / kGRows);
+    p.ksplit = 1;
+    p.kb_part = p.k_blocks;
+    bool wide = false;
     const int limit = c.gated ? 128 : 256;
     if (c.experts) {
         // expected tokens per expert decide the tile; an expert with more takes several tiles
@@ -774,8 +814,15 @@ int launch_gemm_tc(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
         size_t nt = (each + each / 2 + 15) / 16 * 16;
         p.nt = static_cast<int>(nt < 32 ? 32 : nt > static_cast<size_t>(limit) ? limit : nt);
     } else {
-        p.nt = choose_tokens(c.m, p.row_tiles, limit, ctx->sm_count);
+        const TileShape t = choose_tile(c.m, c.out_rows, p.k_blocks, c.gated, ctx->sm_count);
+        p.nt = t.nt;
+        p.ksplit = t.ksplit;
+        p.kb_part = (p.k_blocks + t.ksplit - 1) / t.ksplit;
+        wide = t.wide;
     }
+    p.tile_rows = wide && !c.gated ? 2 * kGRows : kGRows;
+    p.box2_row = c.gated ? static_cast<int>(c.up_row) : kGRows;
+    p.row_tiles = static_cast<int>((c.out_rows + p.tile_rows - 1) / p.tile_rows);
     p.token_tiles = static_cast<int>((c.m + p.nt - 1) / p.nt);
     p.tiles = p.row_tiles * p.token_tiles;
     p.experts = c.experts;
@@ -784,19 +831,6 @@ int launch_gemm_tc(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
     p.err_word = ctx->err_word;
     LBK_TRY(encode_bytes_map(&p.w, c.w.w, c.w.pitch * 2, c.w.rows, c.w.pitch * 2, 128, kGRows));
     LBK_TRY(encode_bytes_map(&p.x, c.x, c.w.pitch * 2, c.m, static_cast<size_t>(c.ldx) * 2, 128, p.nt));
-    // K split over a cluster: at most kGSplitCtas CTAs in all (clusters live inside a GPC, so not every SM can be part
-    // of one), at least four K blocks each
-    p.ksplit = 1;
-    p.kb_part = p.k_blocks;
-    if (!c.experts)
-        for (int s = 8; s >= 2; s >>= 1) {
-            const int part = (p.k_blocks + s - 1) / s;
-            if (p.tiles * s <= kGSplitCtas && part >= 4 && part * (s - 1) < p.k_blocks && p.nt * (c.gated ? 2 : 1) * kGRows * 4 <= kGBars) {
-                p.ksplit = s;
-                p.kb_part = part;
-                break;
-            }
-        }
     if (p.ksplit > 1) {
         cudaLaunchConfig_t cfg{};
         cfg.gridDim = dim3(static_cast<unsigned>(p.tiles * p.ksplit));
@@ -811,10 +845,12 @@ int launch_gemm_tc(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
         attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
         cfg.attrs = attr;
         cfg.numAttrs = 2;
-        LBK_CUDA(cudaLaunchKernelEx(&cfg, c.gated ? dense_gemm_kernel<true, true> : dense_gemm_kernel<false, true>, p));
+        LBK_CUDA(cudaLaunchKernelEx(&cfg, c.gated ? dense_gemm_kernel<kGated, true> : dense_gemm_kernel<0, true>, p));
     } else {
         const int grid = !c.experts && p.tiles < ctx->sm_count ? p.tiles : ctx->sm_count;
-        LBK_CUDA(launch_chained(c.gated ? dense_gemm_kernel<true, false> : dense_gemm_kernel<false, false>, dim3(static_cast<unsigned>(grid)), dim3(kGThreads),
+        void (*k)(GemmParams) = wide ? (c.gated ? dense_gemm_kernel<kGated | kWide, false> : dense_gemm_kernel<kWide, false>)
+                                     : (c.gated ? dense_gemm_kernel<kGated, false> : dense_gemm_kernel<0, false>);
+        LBK_CUDA(launch_chained(k, dim3(static_cast<unsigned>(grid)), dim3(kGThreads),
                                 static_cast<size_t>(kGSmem), st, p));
     }
     LBK_CUDA(cudaGetLastError());
@@ -849,16 +885,13 @@ int dense_init(Ctx *ctx) {
     constexpr size_t parts = static_cast<size_t>(2 * kFewMaxCtas) * kFewPart * sizeof(float) + kFewMaxTiles * sizeof(int);
     LBK_CUDA(cudaMalloc(&ctx->few_parts, parts));
     LBK_CUDA(cudaMemset(ctx->few_parts, 0, parts));
-    const int few_max = 2 * kFewWarps * 2 * 2 * 128 * 4 + static_cast<int>(kFewXSmem);
-    LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
-    LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
-    LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
-    LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
+    const int few_max = 2 * kFewWarps * 2 * 128 * 4 + static_cast<int>(kFewXSmem);
+    LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
+    LBK_CUDA(cudaFuncSetAttribute(dense_few_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, few_max));
     if (static_cast<size_t>(kGSmem) > ctx->smem_optin) return fail(LBK_ERR_UNSUPPORTED, "dense GEMM kernel needs %d B of shared memory", kGSmem);
-    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
-    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
-    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
-    LBK_CUDA(cudaFuncSetAttribute(dense_gemm_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
+    for (void (*k)(GemmParams) : {dense_gemm_kernel<0, false>, dense_gemm_kernel<kGated, false>, dense_gemm_kernel<kWide, false>,
+                                  dense_gemm_kernel<kGated | kWide, false>, dense_gemm_kernel<0, true>, dense_gemm_kernel<kGated, true>})
+        LBK_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kGSmem));
     return LBK_OK;
 }
 const InitHook kInitDense(dense_init);
@@ -872,7 +905,7 @@ int launch_dense(Ctx *ctx, const DenseCall &c, cudaStream_t st) {
     if (!c.w.w || (!c.x && c.pre.mode == kPreNone)) return fail(LBK_ERR_INVALID, "dense projection: null buffer");
     if (c.compute == LBK_COMPUTE_F32) return launch_f32(ctx, c, st);
     if (c.pre.mode != kPreNone && (!dense_pre_supported(c.m, c.w.cols) || c.experts)) return fail(LBK_ERR_INVALID, "dense projection: this call cannot run the norms itself");
-    if (c.m <= LBK_GEMV_MAX_M && !c.experts) return launch_few(ctx, c, st);
+    if (c.m <= static_cast<size_t>(kFewTokens) && !c.experts) return launch_few(ctx, c, st);
     return launch_gemm_tc(ctx, c, st);
 }
 

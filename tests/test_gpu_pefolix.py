@@ -180,6 +180,27 @@ def test_unequal_requests_share_a_cache(nets, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", list(TOL))
+@pytest.mark.parametrize("b", [9, 16])
+def test_large_batches(nets, dtype, b):
+    """Nine and sixteen sequences (other projection kernels than up to eight), every position different."""
+    import torch
+    cfg, _, models = nets["wide"]
+    net = models[dtype]
+    seqs = [tokens(400 + s, 3 + 11 * s + 4, cfg["vocab"]) for s in range(b)]
+    c = net.new_cache(b, 190)
+    for s in range(b):
+        net.forward_rows(seqs[s][:-4], c, [], seq=s)
+    rows = [[] for _ in range(b)]
+    for i in range(4):
+        lg, _ = net.decode(torch.tensor([int(q[len(q) - 4 + i]) for q in seqs], dtype=torch.int32, device="cuda"), c)
+        for s, r in enumerate(lg.cpu().numpy()):
+            rows[s].append(r)
+    got = np.concatenate([np.stack(r) for r in rows])
+    close(got, np.concatenate([logits(nets, "wide", q)[-4:] for q in seqs]), dtype)
+    net.ctx.check_device_error()
+
+
+@pytest.mark.parametrize("dtype", list(TOL))
 def test_a_used_cache_is_as_good_as_a_new_one(nets, dtype):
     """The same request in a fresh cache and in one that a longer request has left: the same bits."""
     cfg, _, models = nets["wide"]

@@ -91,6 +91,25 @@ def test_dense_linear(ctx, po, compute, rows, cols):
     ctx.check_device_error()
 
 
+@pytest.mark.parametrize("rows,cols,m,gated", [(5000, 1024, 2053, 0), (2500, 4096, 2053, 1), (2560, 6912, 2048, 0), (300, 4096, 2000, 1), (129, 8192, 40, 0)])
+def test_dense_linear_large(ctx, rows, cols, m, gated):
+    """Sizes at which the tile shapes change (two weight boxes a tile, K split over a cluster), ragged in rows and tokens,
+    against a 32-bit product of the same values."""
+    import torch
+    L, lib = _lib()
+    torch.manual_seed(rows)
+    x = torch.randn(m, cols, device="cuda").to(torch.bfloat16)
+    w = (torch.randn(rows * (2 if gated else 1), cols, device="cuda") * cols ** -0.5).to(torch.bfloat16)
+    out = torch.full((m, pad64(rows)), 7.0, dtype=torch.bfloat16 if gated else torch.float32, device="cuda")
+    L.check(lib.lbk_dense_linear(ctx.handle, BF16, x.data_ptr(), cols, m, w.data_ptr(), cols, w.shape[0], cols, gated, rows, 0, out.data_ptr(),
+                                 out.shape[1], 0 if gated else 1, None, 0, _st()))
+    v = x.float() @ w.float().T
+    want = torch.nn.functional.gelu(v[:, :rows], approximate="tanh") * v[:, rows:] if gated else v
+    assert float((out[:, :rows].float() - want).abs().max()) <= (2.0 ** -8 if gated else 2e-5) * float(want.abs().max())
+    assert bool((out[:, rows:] == 7.0).all())
+    ctx.check_device_error()
+
+
 @pytest.mark.parametrize("compute", [BF16, F32])
 @pytest.mark.parametrize("counts", [[3, 0, 40, 1, 300, 0, 17], [0, 0, 5], [130], [64, 64, 64, 64, 1]])
 def test_dense_linear_of_sorted_tokens(ctx, compute, counts):
