@@ -19,8 +19,9 @@ FAMILIES = {
     "": ["lbk_api.cu", "lbk_gemv.cu", "lbk_quant.cu", "lbk_plan.cu", "lbk_sweep.cu", "lbk_gemm.cu", "lbk_noalloc.cu", "lbk_tp.cu",
          "lbk_bitnet.cu", "lbk_convert.cu", "lbk_probe.cu"],
     "Pefolix": ["lbk_layernorm.cu", "lbk_dense.cu", "lbk_moe.cu", "lbk_attn_window.cu", "lbk_pefolix.cu"],
+    "Dugulorn": ["lbk_layernorm.cu", "lbk_dense.cu", "lbk_attn_window.cu", "lbk_latent.cu", "lbk_recur.cu", "lbk_dugulorn.cu"],
 }
-SOURCES = RUNTIME + [s for f in FAMILIES.values() for s in f]
+SOURCES = RUNTIME + list(dict.fromkeys(s for f in FAMILIES.values() for s in f))  # families share kernel files
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC",

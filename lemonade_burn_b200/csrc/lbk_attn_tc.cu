@@ -36,6 +36,10 @@
 // kept first tokens, then those some row's window reaches), the distance bias taken off the f32 scores, and a
 // bf16 output. A row may see nothing of a block then, so its maximum starts at a finite value.
 //
+// The two-part form (FORM = kTwoPart) is the windowed one with longer keys: a key is a part of the head's own (dimp) and a
+// part all heads share (dim2p, from rows of another buffer), each in pieces of 64 dimensions, three pieces in all, and
+// only two K blocks in the ring; the output may be multiplied by a gate per row and head.
+//
 // Rows of V past the keys written so far may hold anything (they are multiplied by exact zeros,
 // and 0 * NaN is NaN): the block that reaches past them has them zeroed in shared memory first.
 #include "lbk_dense.cuh"
@@ -67,6 +71,10 @@ constexpr int kThreads = 10 * 32;
 constexpr uint32_t kTmemCols = 512;
 constexpr uint32_t kColS = 0, kColO = 128, kColP = 256;  // P buffer b: hi at kColP + 128 b, lo 64 columns further
 constexpr float kRescaleStep = 8.0f;        // in units of log 2
+constexpr int kPlain = 0, kWindow = 1, kTwoPart = 2;
+// two-part keys: Q three pieces, two K blocks of three pieces
+constexpr int kTpPieces = 3, kTpKStages = 2, kTpK0 = kTpPieces * kHalf, kTpV0 = kTpK0 + kTpKStages * kTpPieces * kHalf;
+static_assert(kTpV0 + kVStages * kBlockBytes <= kBars, "two-part keys: shared memory budget");
 
 struct AttnParams {
     CUtensorMap k, v;     // bytes [cache rows][256], box [128][128], SWIZZLE_128B
@@ -82,6 +90,11 @@ struct AttnParams {
     long ldo;
     int dimp, vdim, vdimp, win, keep;
     float slope_unit;     // head h: log2(e) * 2^(-8 (h + 1) / nh), or 0
+    // two-part keys
+    CUtensorMap k2;       // bytes [positions][dim2p * 2]
+    int dim2p;
+    const float *gate;    // logits [n][ldg], or null
+    long ldg;
 };
 
 using dense::bf16_pair;
@@ -127,8 +140,10 @@ __device__ __forceinline__ void umma_f16_ts(uint32_t d_tmem, uint32_t a_tmem, ui
                  : "memory");
 }
 
-template <bool WINDOW>
+template <int FORM>
 __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __grid_constant__ AttnParams p) {
+    constexpr bool WINDOW = FORM != kPlain, TWO = FORM == kTwoPart;
+    constexpr int kKStages = TWO ? kTpKStages : lbk::kKStages, kKBytes = (TWO ? kTpPieces : 2) * kHalf, kK0 = TWO ? kTpK0 : lbk::kK0, kV0 = TWO ? kTpV0 : lbk::kV0;
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw = ptx::smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
@@ -187,7 +202,20 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
     if (warp < kSoftWarps) {
         const int r = (warp & 3) * 32 + lane;
         const bool live = r < rows_here && pos_ok;
-        if (WINDOW) {
+        if (TWO) {
+            const uint16_t *qr = p.q16 + (static_cast<size_t>(row0 + (live ? r : 0)) * p.nh + head) * (p.dimp + p.dim2p);
+            const int n1 = (p.dimp + 63) >> 6, n2 = (p.dim2p + 63) >> 6;
+            for (int piece = 0; piece < n1 + n2; ++piece) {
+                const int d0 = piece < n1 ? piece * 64 : (piece - n1) * 64, end = piece < n1 ? p.dimp : p.dim2p, from = piece < n1 ? 0 : p.dimp;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int u = (warp >> 2) * 4 + e;
+                    uint4 a = make_uint4(0u, 0u, 0u, 0u);
+                    if (live && d0 + u * 8 < end) a = *reinterpret_cast<const uint4 *>(qr + from + d0 + u * 8);
+                    *reinterpret_cast<uint4 *>(sm + piece * kHalf + r * 128 + ((u ^ (r & 7)) << 4)) = a;
+                }
+            }
+        } else if (WINDOW) {
             const uint16_t *qr = p.q16 + (static_cast<size_t>(row0 + (live ? r : 0)) * p.nh + head) * p.dimp;
 #pragma unroll 4
             for (int u = (warp >> 2) * 8; u < (warp >> 2) * 8 + 8; ++u) {
@@ -234,11 +262,18 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
                     ok = false;
                     break;
                 }
-                const uint32_t kst = base + kK0 + ks * kBlockBytes;
+                const uint32_t kst = base + kK0 + ks * kKBytes;
                 const bool k2 = !WINDOW || p.dimp > 64, v2 = !WINDOW || p.vdimp > 64;  // a second half of 64 dimensions
-                ptx::mbar_arrive_expect_tx(bar(kKFull + ks), k2 ? kBlockBytes : kHalf);
-                ptx::tma_load_2d(kst, &p.k, bar(kKFull + ks), 0, y);
-                if (k2) ptx::tma_load_2d(kst + kHalf, &p.k, bar(kKFull + ks), 128, y);
+                if (TWO) {
+                    const int n1 = (p.dimp + 63) >> 6, n2 = (p.dim2p + 63) >> 6;
+                    ptx::mbar_arrive_expect_tx(bar(kKFull + ks), (n1 + n2) * kHalf);
+                    for (int piece = 0; piece < n1; ++piece) ptx::tma_load_2d(kst + piece * kHalf, &p.k, bar(kKFull + ks), piece * 128, y);
+                    for (int piece = 0; piece < n2; ++piece) ptx::tma_load_2d(kst + (n1 + piece) * kHalf, &p.k2, bar(kKFull + ks), piece * 128, block_of(j) * kTile);
+                } else {
+                    ptx::mbar_arrive_expect_tx(bar(kKFull + ks), k2 ? kBlockBytes : kHalf);
+                    ptx::tma_load_2d(kst, &p.k, bar(kKFull + ks), 0, y);
+                    if (k2) ptx::tma_load_2d(kst + kHalf, &p.k, bar(kKFull + ks), 128, y);
+                }
                 if (++ks == kKStages) {
                     ks = 0;
                     ++kround;
@@ -265,7 +300,15 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
             const uint64_t q_desc = smem_desc_sw128(base);
             int ks = 0, kphase = 0;  // ring position of the K block the next Q K^T reads
             auto issue_s = [&]() {   // S = Qhi K^T + Qlo K^T over the 8 steps of 16 dimensions
-                const uint64_t k_desc = smem_desc_sw128(base + kK0 + ks * kBlockBytes);
+                const uint64_t k_desc = smem_desc_sw128(base + kK0 + ks * kKBytes);
+                if (TWO) {
+                    const int n1 = (p.dimp + 63) >> 6, s2 = p.dim2p >> 4;
+                    for (int st = 0; st < dim_steps + s2; ++st) {
+                        const int in = st < dim_steps ? st : st - dim_steps, piece = (st < dim_steps ? 0 : n1) + (in >> 2);
+                        const uint64_t off = static_cast<uint64_t>(piece * (kHalf >> 4) + (in & 3) * 2);
+                        umma_f16_ss(tmem_base + kColS, q_desc + off, k_desc + off, idesc_s, st ? 1u : 0u);
+                    }
+                } else
 #pragma unroll
                 for (int t = 0; t < (WINDOW ? 1 : 2); ++t)
 #pragma unroll
@@ -449,7 +492,8 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
         pair_sync();
         const float lsum = pair_l[r] + pair_l[kTile + r];
         if (ok && nb > 0) {
-            const float inv = 1.0f / lsum;
+            float inv = 1.0f / lsum;
+            if (TWO && p.gate && r < rows_here) inv *= dense::sigmoid(p.gate[static_cast<size_t>(row0 + r) * p.ldg + head]);
             float *dst = WINDOW ? nullptr : p.out + (static_cast<size_t>(row0 + (r < rows_here ? r : 0)) * p.nh + head) * kHd + kh2 * 64;
 #pragma unroll 1
             for (int c = 0; c < 2; ++c) {  // this warp's 64 dimensions of the row
@@ -504,8 +548,8 @@ __global__ void __launch_bounds__(kThreads, 1) attn_prompt_tc_kernel(const __gri
 
 int attn_tc_init(Ctx *ctx) {
     if (static_cast<size_t>(kSmem) > ctx->smem_optin) return fail(LBK_ERR_UNSUPPORTED, "prompt attention kernel needs %d B of shared memory", kSmem);
-    LBK_CUDA(cudaFuncSetAttribute(attn_prompt_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
-    LBK_CUDA(cudaFuncSetAttribute(attn_prompt_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+    for (void (*k)(AttnParams) : {attn_prompt_tc_kernel<kPlain>, attn_prompt_tc_kernel<kWindow>, attn_prompt_tc_kernel<kTwoPart>})
+        LBK_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
     return LBK_OK;
 }
 static const InitHook kInitAttnTc(attn_tc_init);
@@ -527,7 +571,7 @@ int launch_attn_prompt_tc(Ctx *ctx, const float *q, const uint16_t *kc, const ui
     p.scaling = 1.4426950408889634f / sqrtf(static_cast<float>(kHd));  // scores in units of log 2: the softmax is 2^(s - max)
     p.err_word = ctx->err_word;
     const dim3 grid(static_cast<unsigned>(nh), static_cast<unsigned>((n + kTile - 1) / kTile));
-    LBK_CUDA(launch_chained(attn_prompt_tc_kernel<false>, grid, dim3(kThreads), static_cast<size_t>(kSmem), stream, p));
+    LBK_CUDA(launch_chained(attn_prompt_tc_kernel<kPlain>, grid, dim3(kThreads), static_cast<size_t>(kSmem), stream, p));
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;
     return LBK_OK;
@@ -536,7 +580,15 @@ int launch_attn_prompt_tc(Ctx *ctx, const float *q, const uint16_t *kc, const ui
 int launch_attn_window_tc(Ctx *ctx, const AttnCall &c, cudaStream_t stream) {
     if (c.dimp > 128 || c.vdimp > 128 || c.dimp % 16 || c.vdimp % 16 || c.rows_of_seq < 0 || c.ldo % 8)
         return fail(LBK_ERR_INVALID, "windowed prompt attention: padded head sizes are multiples of 16, at most 128");
+    if (c.k2 && ((c.dimp + 63) / 64 + (c.dim2p + 63) / 64 > static_cast<size_t>(kTpPieces) || c.dim2p % 16 || c.k2_pitch % 8))
+        return fail(LBK_ERR_INVALID, "prompt attention with two-part keys: three pieces of 64 dimensions at most");
     AttnParams p{};
+    if (c.k2) {
+        LBK_TRY(encode_bytes_map(&p.k2, c.k2, c.dim2p * 2, c.k2_rows, c.k2_pitch * 2, 128, kTile));
+        p.dim2p = static_cast<int>(c.dim2p);
+        p.gate = c.gate;
+        p.ldg = c.ldg;
+    }
     const size_t cache_rows = static_cast<size_t>(c.rows_of_seq + 1) * c.kv_heads * c.cap;
     LBK_TRY(encode_bytes_map(&p.k, c.kc, c.dimp * 2, cache_rows, c.dimp * 2, 128, kTile));
     LBK_TRY(encode_bytes_map(&p.v, c.vc, c.vdimp * 2, cache_rows, c.vdimp * 2, 128, kTile));
@@ -558,7 +610,7 @@ int launch_attn_window_tc(Ctx *ctx, const AttnCall &c, cudaStream_t stream) {
     p.keep = c.mask.keep_first;
     p.slope_unit = c.mask.alibi ? 1.4426950408889634f : 0.0f;
     const dim3 grid(static_cast<unsigned>(c.heads), static_cast<unsigned>((c.n + kTile - 1) / kTile));
-    LBK_CUDA(launch_chained(attn_prompt_tc_kernel<true>, grid, dim3(kThreads), static_cast<size_t>(kSmem), stream, p));
+    LBK_CUDA(launch_chained(c.k2 ? attn_prompt_tc_kernel<kTwoPart> : attn_prompt_tc_kernel<kWindow>, grid, dim3(kThreads), static_cast<size_t>(kSmem), stream, p));
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;
     return LBK_OK;

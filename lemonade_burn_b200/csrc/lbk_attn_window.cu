@@ -11,7 +11,7 @@
 //                              of one mma.sync tile (16 at a time), visible keys in slices of whole 64-key chunks,
 //                              two stages of cp.async; scores, probabilities (two bf16 terms) and sums in f32.
 //   attn_window_combine_kernel merges the slices.
-//   attn_window_kernel         any head size up to 512, bf16 or f32, any rows: one block per (row, head). The
+//   attn_window_kernel         any head size up to 512 (f32: 1024), bf16 or f32, any rows: one block per (row, head). The
 //                              32-bit path, portions of a few rows, and head sizes the others do not have.
 // Prompt rows go to the tcgen05 kernel in lbk_attn_tc.cu.
 #include "lbk_dense.cuh"
@@ -368,7 +368,7 @@ __global__ void __launch_bounds__(128) attn_window_combine_kernel(const WinParam
     }
 }
 
-constexpr size_t kMaxDim = 512;
+constexpr size_t kMaxDim = 512, kMaxDim32 = 1024;  // 16-bit, 32-bit
 constexpr size_t kTcMinRows = 8;  // prompt rows from which the 128-row tiles of the tcgen05 kernel are worth it
 
 template <typename T>
@@ -377,7 +377,8 @@ int launch_generic(Ctx *ctx, const WinParams &p, cudaStream_t st) {
     const int d = p.dim > p.vdim ? p.dim : p.vdim;
     if (d <= 128) LBK_CUDA(launch_chained(attn_window_kernel<T, 4>, grid, dim3(128), 0, st, p));
     else if (d <= 256) LBK_CUDA(launch_chained(attn_window_kernel<T, 8>, grid, dim3(128), 0, st, p));
-    else LBK_CUDA(launch_chained(attn_window_kernel<T, 16>, grid, dim3(128), 0, st, p));
+    else if (d <= 512) LBK_CUDA(launch_chained(attn_window_kernel<T, 16>, grid, dim3(128), 0, st, p));
+    else LBK_CUDA(launch_chained(attn_window_kernel<T, sizeof(T) == 4 ? 32 : 16>, grid, dim3(128), 0, st, p));
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;
     return LBK_OK;
@@ -411,7 +412,8 @@ int launch_attn_window(Ctx *ctx, const AttnCall &c, cudaStream_t st) {
     if (!c.q || !c.kc || !c.vc || !c.pos || !c.out) return fail(LBK_ERR_INVALID, "windowed attention: null buffer");
     if (c.kv_heads == 0 || c.heads % c.kv_heads || c.dim == 0 || c.vdim == 0 || c.dim > c.dimp || c.vdim > c.vdimp || c.dimp % 16 || c.vdimp % 16)
         return fail(LBK_ERR_SHAPE, "windowed attention: inconsistent head counts or sizes");
-    if (c.dim > kMaxDim || c.vdim > kMaxDim) return fail(LBK_ERR_UNSUPPORTED, "windowed attention: head sizes of at most %zu", kMaxDim);
+    const size_t most = c.compute == LBK_COMPUTE_F32 ? kMaxDim32 : kMaxDim;
+    if (c.dim > most || c.vdim > most) return fail(LBK_ERR_UNSUPPORTED, "windowed attention: head sizes of at most %zu", most);
     if (c.n > 65535) return fail(LBK_ERR_UNSUPPORTED, "at most 65535 rows per call");
     WinParams p{};
     p.q = c.q;

@@ -82,7 +82,7 @@ __device__ __forceinline__ void few_norm_row(const FewParams &p, int t, bool wri
             v[j] = i < n4 ? yr[i] : zero;
             s += (v[j].x + v[j].y) + (v[j].z + v[j].w);
         }
-        const float mean = dense::block_sum<kFewThreads>(s, s_red) * inv_n;
+        const float mean = p.pre.rms ? 0.0f : dense::block_sum<kFewThreads>(s, s_red) * inv_n;
         float ss = 0.0f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -101,25 +101,31 @@ __device__ __forceinline__ void few_norm_row(const FewParams &p, int t, bool wri
             }
         }
     }
-    float s = 0.0f;
+    float r = 1.0f;
+    if (p.pre.w) {
+        float mean = 0.0f;
+        if (!p.pre.rms) {
+            float s = 0.0f;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) s += (u[j].x + u[j].y) + (u[j].z + u[j].w);
-    const float mean = dense::block_sum<kFewThreads>(s, s_red) * inv_n;
-    float ss = 0.0f;
+            for (int j = 0; j < 4; ++j) s += (u[j].x + u[j].y) + (u[j].z + u[j].w);
+            mean = dense::block_sum<kFewThreads>(s, s_red) * inv_n;
+        }
+        float ss = 0.0f;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-        const int i = tid + j * kFewThreads;
-        u[j] = i < n4 ? make_float4(u[j].x - mean, u[j].y - mean, u[j].z - mean, u[j].w - mean) : zero;
-        ss += (u[j].x * u[j].x + u[j].y * u[j].y) + (u[j].z * u[j].z + u[j].w * u[j].w);
+        for (int j = 0; j < 4; ++j) {
+            const int i = tid + j * kFewThreads;
+            u[j] = i < n4 ? make_float4(u[j].x - mean, u[j].y - mean, u[j].z - mean, u[j].w - mean) : zero;
+            ss += (u[j].x * u[j].x + u[j].y * u[j].y) + (u[j].z * u[j].z + u[j].w * u[j].w);
+        }
+        r = 1.0f / sqrtf(dense::block_sum<kFewThreads>(ss, s_red) * inv_n + p.pre.eps);
     }
-    const float r = 1.0f / sqrtf(dense::block_sum<kFewThreads>(ss, s_red) * inv_n + p.pre.eps);
     const int pad4 = p.chunks * 8;          // chunks of 32 columns: zeros past the row
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
         const int i = tid + j * kFewThreads;
         uint2 o = make_uint2(0u, 0u);
         if (i < n4) {
-            const float4 g = __ldg(reinterpret_cast<const float4 *>(p.pre.w) + i);
+            const float4 g = p.pre.w ? __ldg(reinterpret_cast<const float4 *>(p.pre.w) + i) : make_float4(1.f, 1.f, 1.f, 1.f);
             o = make_uint2(dense::bf16_pair(u[j].x * r * g.x, u[j].y * r * g.y), dense::bf16_pair(u[j].z * r * g.z, u[j].w * r * g.w));
             if (writer && p.pre.nout) reinterpret_cast<uint2 *>(static_cast<uint16_t *>(p.pre.nout) + static_cast<size_t>(t) * p.pre.ldn)[i] = o;
         }

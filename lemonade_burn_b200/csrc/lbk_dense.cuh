@@ -11,8 +11,9 @@ struct DenseWeight {
     size_t rows = 0, cols = 0, pitch = 0;
 };
 inline size_t dense_pitch(size_t cols) { return (cols + 63) / 64 * 64; }
+inline size_t pad16(size_t v) { return (v + 15) / 16 * 16; }
 
-constexpr int kActNone = 0, kActRelu2 = 1;
+constexpr int kActNone = 0, kActRelu2 = 1, kActSilu = 2;
 constexpr int kEpiF32 = 0;   // f32 rows: out[t * ld + r]
 constexpr int kEpiElem = 1;  // act(v) in the compute type; rows from f32_from on as f32 into out2[t * ld2 + r - f32_from]
 constexpr int kEpiQkv = 2;   // rows of a stacked [q; k; v] projection: q to its buffer, k and v into the cache at the token's position
@@ -20,6 +21,8 @@ constexpr int kEpiQkv = 2;   // rows of a stacked [q; k; v] projection: q to its
 // What happens to the value of (token t, output row r).
 struct DenseEpi {
     int kind = kEpiF32, act = kActNone;
+    int act_rows = 1 << 30;      // kEpiElem: output rows below this one get the activation
+    const float *bias = nullptr; // [out_rows], added first (not with gated)
     void *out = nullptr;
     long ld = 0;
     int f32_from = 1 << 30;
@@ -27,6 +30,7 @@ struct DenseEpi {
     long ld2 = 0;
     // kEpiQkv: q [t][heads][dimp] in `out` (ld = heads * dimp); caches [seq][kv_heads][cap][dimp / vdimp]
     int q_rows = 0, k_rows = 0, dim = 1, dimp = 1, vdim = 1, vdimp = 1, kv_heads = 1, cap = 0;
+    int q_split = 1 << 30, q_gap = 0;  // dimensions of a q head from q_split on go q_gap places further
     void *kc = nullptr, *vc = nullptr;
     const int *pos = nullptr;  // decode: one position per token (= sequence); rows: pos[0] is the first token's
     int rows_of_seq = -1;      // >= 0: the tokens are consecutive positions of this sequence; -1: token t is sequence t
@@ -36,9 +40,10 @@ struct DenseEpi {
 // The norms in front of a projection, done inside the few-row kernel (kPreNone: the input rows are ready).
 constexpr int kPreNone = 0;
 constexpr int kPreNorm = 1;     // n = norm(x) * w
-constexpr int kPreAddNorm = 2;  // s = x + norm(y) * w_post (written to xout), n = norm(s) * w
+constexpr int kPreAddNorm = 2;  // s = x + norm(y) * w_post (written to xout), n = norm(s) * w (w null: n = s)
 struct DensePre {
     int mode = kPreNone;
+    bool rms = false;           // the norms divide by the root mean square, without taking the mean off
     const float *x = nullptr, *y = nullptr, *w_post = nullptr, *w = nullptr;
     float *xout = nullptr;
     void *nout = nullptr;  // optional: the normalised rows in the compute type, pitch ldn
@@ -87,16 +92,22 @@ struct AttnCall {
     float *scratch = nullptr; // decode: attn_window_scratch floats
     void *out = nullptr;      // [rows][heads * vdim] of the compute type, pitch ldo
     long ldo = 0;
+    // prompt rows on tcgen05 only: a second part of every key, the same for all heads (rows of k2_pitch values by
+    // position); a query head is [dimp | dim2p] then. And a gate per row and head: the output times sigmoid(gate).
+    const void *k2 = nullptr;
+    size_t dim2p = 0, k2_pitch = 0, k2_rows = 0;
+    const float *gate = nullptr;
+    long ldg = 0;
 };
 size_t attn_window_scratch(size_t b, size_t heads, size_t vdimp, size_t splits);
 size_t attn_window_splits(size_t cap, const AttnMask &mask);
 int launch_attn_window(Ctx *ctx, const AttnCall &c, cudaStream_t st);
-// the tcgen05 form of it for prompt rows (lbk_attn_tc.cu); bf16, dim and vdim at most 128
+// the tcgen05 form of it for prompt rows (lbk_attn_tc.cu); bf16, dim and vdim at most 128 (with k2: three pieces of 64)
 int launch_attn_window_tc(Ctx *ctx, const AttnCall &c, cudaStream_t st);
 
 // ---- norms (lbk_layernorm.cu) -------------------------------------------------------------------
-// x += norm(y) * w_post (y null: x as it is); then n = norm(x) * w to out_f (f32, pitch n) and / or out_e
-// (compute type, pitch lde). w null: only the sum. The sublayer's rows are y, or with `moe` the expert outputs.
+// x += norm(y) * w_post (y null: x as it is); then n = norm(x) * w to out_f (f32, pitch n; may be x itself) and / or
+// out_e (compute type, pitch lde). w null: n is the sum itself. norm: layer norm, or with `rms` the RMS norm. The sublayer's rows are y, or with `moe` the expert outputs.
 struct MoeOut {
     const uint16_t *rows16 = nullptr;  // expert outputs by sorted row, bf16 or f32, pitch ld
     const float *rows32 = nullptr;
@@ -109,6 +120,7 @@ struct MoeOut {
 };
 struct NormCall {
     int compute = LBK_COMPUTE_BF16;
+    bool rms = false;
     float *x = nullptr;
     const float *y = nullptr, *w_post = nullptr, *w = nullptr;
     const MoeOut *moe = nullptr;

@@ -38,6 +38,13 @@ __device__ __forceinline__ float relu2(float z) {
     return r * r;
 }
 
+// z / (1 + e^-z); e^-z overflows to inf for large negative z: -0
+template <bool EXACT>
+__device__ __forceinline__ float silu(float z) {
+    if (EXACT) return z / (1.0f + expf(-z));
+    return z * __frcp_rn(1.0f + __expf(-z));
+}
+
 // Sum over the block; every thread gets it. `s_red`: 32 floats, may be reused right away.
 template <int NT>
 __device__ __forceinline__ float block_sum(float v, float *s_red) {
@@ -55,6 +62,7 @@ __device__ __forceinline__ float block_sum(float v, float *s_red) {
 // Where output row r of a call goes, worked out once per row; the token is added per store.
 struct RowPlan {
     int mode = 0;  // 0: drop, 1: f32, 2: compute type with the activation, 3: compute type
+    float bias = 0.0f;
     char *base = nullptr;
     long stride = 0, seq_stride = 0;
     bool by_pos = false;
@@ -62,6 +70,7 @@ struct RowPlan {
 template <typename T>
 __device__ __forceinline__ RowPlan row_plan(const DenseEpi &e, int r, int pos0) {
     RowPlan q;
+    if (e.bias) q.bias = e.bias[r];
     if (e.kind == kEpiF32) {
         q.mode = 1;
         q.base = reinterpret_cast<char *>(static_cast<float *>(e.out) + r);
@@ -72,7 +81,7 @@ __device__ __forceinline__ RowPlan row_plan(const DenseEpi &e, int r, int pos0) 
             q.base = reinterpret_cast<char *>(e.out2 + (r - e.f32_from));
             q.stride = e.ld2;
         } else {
-            q.mode = 2;
+            q.mode = r < e.act_rows ? 2 : 3;
             q.base = reinterpret_cast<char *>(static_cast<T *>(e.out) + r);
             q.stride = e.ld;
         }
@@ -80,7 +89,7 @@ __device__ __forceinline__ RowPlan row_plan(const DenseEpi &e, int r, int pos0) 
         q.mode = 3;
         if (r < e.q_rows) {
             const int h = r / e.dim, d = r - h * e.dim;
-            q.base = reinterpret_cast<char *>(static_cast<T *>(e.out) + h * e.dimp + d);
+            q.base = reinterpret_cast<char *>(static_cast<T *>(e.out) + h * e.dimp + d + (d >= e.q_split ? e.q_gap : 0));
             q.stride = e.ld;
         } else {
             const bool is_k = r < e.q_rows + e.k_rows;
@@ -111,8 +120,9 @@ __device__ __forceinline__ void row_store(const DenseEpi &e, const RowPlan &q, i
         }
         off = static_cast<long>(t) * q.seq_stride + static_cast<long>(pos) * q.stride;
     }
+    v += q.bias;
     if (q.mode == 1) reinterpret_cast<float *>(q.base)[off] = v;
-    else if (q.mode == 2) put(reinterpret_cast<T *>(q.base) + off, e.act == kActRelu2 ? relu2(v) : v);
+    else if (q.mode == 2) put(reinterpret_cast<T *>(q.base) + off, e.act == kActRelu2 ? relu2(v) : e.act == kActSilu ? silu<sizeof(T) == 4>(v) : v);
     else if (q.mode == 3) put(reinterpret_cast<T *>(q.base) + off, v);
 }
 // A prompt pass whose positions do not fit the cache must not store anything.

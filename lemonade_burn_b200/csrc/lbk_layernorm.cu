@@ -1,10 +1,11 @@
 // Layer norm with a weight and no bias, (x - mean) / sqrt(var + eps) * w with var the mean of the squared
-// deviations, and the "sandwich" step around a sublayer: the sublayer's output is normalised before it joins the
+// deviations, or RMS norm, x / sqrt(mean(x^2) + eps) * w, and the "sandwich" step around a sublayer: the sublayer's output is normalised before it joins the
 // f32 residual, and the next sublayer's input is the norm of the sum. One kernel does all of it for a row:
 //
 //     x += norm(y) * w_post        y: a projection's rows, or the outputs of a token's experts (gathered,
 //                                  weighted and summed here) plus the gated shared expert
-//     n  = norm(x) * w             to f32 (the head's input) and / or the compute type (a projection's input)
+//     n  = norm(x) * w             to f32 (the head's input) and / or the compute type (a projection's input);
+//                                  without w the sum itself (sublayers that read the residual un-normed)
 //
 // The row stays in registers between the four reductions (up to 8192 values at 256 threads a row; longer rows
 // take 1024 threads).
@@ -20,7 +21,7 @@ struct NormParams {
     float *x;
     const float *y, *w_post, *w;
     MoeOut moe;
-    int has_moe, n;
+    int has_moe, n, rms;
     float eps;
     float *out_f;
     void *out_e;
@@ -64,7 +65,7 @@ __global__ void __launch_bounds__(NT) sandwich_norm_kernel(const NormParams p) {
             v[j] = t;
             s += t;
         }
-        const float mean = dense::block_sum<NT>(s, s_red) * inv_n;
+        const float mean = p.rms ? 0.0f : dense::block_sum<NT>(s, s_red) * inv_n;
         float ss = 0.0f;
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
@@ -88,11 +89,21 @@ __global__ void __launch_bounds__(NT) sandwich_norm_kernel(const NormParams p) {
             v[j] = i < n ? xr[i] : 0.0f;
         }
     }
-    if (!p.w) return;
+    if (!p.w) {  // the sum itself
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + j * NT;
+            if (i < n) {
+                if (p.out_f) p.out_f[row * n + i] = v[j];
+                if (p.out_e) dense::put(static_cast<T *>(p.out_e) + row * p.lde + i, v[j]);
+            }
+        }
+        return;
+    }
     float s = 0.0f;
 #pragma unroll
     for (int j = 0; j < NV; ++j) s += v[j];
-    const float mean = dense::block_sum<NT>(s, s_red) * inv_n;
+    const float mean = p.rms ? 0.0f : dense::block_sum<NT>(s, s_red) * inv_n;
     float ss = 0.0f;
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
@@ -167,7 +178,7 @@ __global__ void __launch_bounds__(256) sandwich_norm_vec_kernel(const NormParams
         }
 #pragma unroll
         for (int j = 0; j < NV; ++j) s += sum4(v[j]);
-        const float mean = dense::block_sum<256>(s, s_red) * inv_n;
+        const float mean = p.rms ? 0.0f : dense::block_sum<256>(s, s_red) * inv_n;
         float ss = 0.0f;
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
@@ -192,11 +203,21 @@ __global__ void __launch_bounds__(256) sandwich_norm_vec_kernel(const NormParams
             v[j] = i < n4 ? xr[i] : zero;
         }
     }
-    if (!p.w) return;
+    if (!p.w) {  // the sum itself
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + j * 256;
+            if (i < n4) {
+                if (p.out_f) reinterpret_cast<float4 *>(p.out_f + row * n)[i] = v[j];
+                if (p.out_e) dense::put4(static_cast<T *>(p.out_e) + row * p.lde + 4 * i, v[j]);
+            }
+        }
+        return;
+    }
     float s = 0.0f;
 #pragma unroll
     for (int j = 0; j < NV; ++j) s += sum4(v[j]);
-    const float mean = dense::block_sum<256>(s, s_red) * inv_n;
+    const float mean = p.rms ? 0.0f : dense::block_sum<256>(s, s_red) * inv_n;
     float ss = 0.0f;
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
@@ -229,6 +250,7 @@ int norm_impl(Ctx *ctx, const NormCall &c, cudaStream_t st) {
     if (c.moe) p.moe = *c.moe;
     p.has_moe = c.moe ? 1 : 0;
     p.n = static_cast<int>(c.n);
+    p.rms = c.rms ? 1 : 0;
     p.eps = c.eps;
     p.out_f = c.out_f;
     p.out_e = c.out_e;

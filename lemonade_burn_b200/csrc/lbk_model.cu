@@ -2,7 +2,7 @@
 // `BitNet::{load, new_cache, forward}` (crates/lb-model/src/model.rs:149-232, 234-236, 305-374) without a
 // tensor framework in between: the registry of model families, the checkpoint file, the cache's slots and
 // positions, the recorded decode step, prompt passes, and the batcher. What a family's step consists of is
-// in its own file (lbk_bitnet.cu, lbk_pefolix.cu).
+// in its own file (lbk_bitnet.cu, lbk_pefolix.cu, lbk_dugulorn.cu).
 //
 // A call with several tokens of one sequence (a prompt, or a portion of one) sends up to 4096 rows at a time
 // through the projections. One decode step is recorded into a CUDA graph the first time a cache is used and
@@ -88,6 +88,75 @@ int TensorFile::find(const std::string &name, const char *dtype, size_t elems, s
         return fail(LBK_ERR_INVALID, "%s is truncated: %s ends at byte %zu, the file has %zu", path.c_str(), name.c_str(), sg.data0 + e.end, sg.file_size);
     *e_out = &e;
     return LBK_OK;
+}
+
+int WeightLoader::shape(const std::string &name, size_t *rows, size_t *cols) const {
+    const auto it = tf.entries.find(name);
+    if (it == tf.entries.end()) return fail(LBK_ERR_INVALID, "%s: tensor %s is missing", tf.path.c_str(), name.c_str());
+    if (it->second.shape.size() != 2) return fail(LBK_ERR_SHAPE, "%s: %s is not a matrix", tf.path.c_str(), name.c_str());
+    *rows = it->second.shape[0];
+    *cols = it->second.shape[1];
+    return LBK_OK;
+}
+
+int WeightLoader::vec(const std::string &name, size_t n, float **out, float add) {
+    const TensorEntry *e;
+    LBK_TRY(tf.find(name, "BF16", n, 2, &e));
+    std::vector<uint16_t> raw(n);
+    if (pread(tf.sg.fd, raw.data(), n * 2, static_cast<off_t>(tf.sg.data0 + e->begin)) != static_cast<ssize_t>(n * 2))
+        return fail(LBK_ERR_INVALID, "cannot read %s", name.c_str());
+    std::vector<float> f(n);
+    for (size_t i = 0; i < n; ++i) {
+        const uint32_t bits = static_cast<uint32_t>(raw[i]) << 16;
+        memcpy(&f[i], &bits, 4);
+        f[i] += add;
+    }
+    tf.sg.bytes_read += n * 2;
+    tf.sg.bytes_to_device += n * 4;
+    return floats(f, out);
+}
+
+int WeightLoader::floats(const std::vector<float> &v, float **out) {
+    LBK_TRY(dev_alloc(owner, v.size() * 4, reinterpret_cast<void **>(out)));
+    LBK_CUDA(cudaMemcpy(*out, v.data(), v.size() * 4, cudaMemcpyHostToDevice));
+    return LBK_OK;
+}
+
+int WeightLoader::stack(const std::vector<std::string> &names, const std::vector<size_t> &rows, size_t cols, DenseWeight *out) {
+    size_t total = 0;
+    bool zeros = false;
+    for (size_t i = 0; i < rows.size(); ++i) {
+        total += rows[i];
+        zeros = zeros || names[i].empty();
+    }
+    const size_t pitch = dense_pitch(cols);
+    uint16_t *dev = nullptr;
+    LBK_TRY(dev_alloc(owner, total * pitch * 2, reinterpret_cast<void **>(&dev)));
+    if (pitch != cols || zeros) LBK_CUDA(cudaMemsetAsync(dev, 0, total * pitch * 2, ctx->own_stream));
+    size_t at = 0;
+    for (size_t i = 0; i < names.size(); ++i) {
+        if (!names[i].empty()) {
+            const TensorEntry *e;
+            LBK_TRY(tf.find(names[i], "BF16", rows[i] * cols, 2, &e));
+            LBK_TRY(tf.sg.copy_rows(e->begin, rows[i], cols * 2, dev + at * pitch, pitch * 2, names[i].c_str()));
+        }
+        at += rows[i];
+    }
+    *out = DenseWeight{dev, total, cols, pitch};
+    return LBK_OK;
+}
+
+int WeightLoader::table(const std::string &name, size_t rows, size_t cols, uint16_t **out) {
+    const TensorEntry *e;
+    LBK_TRY(tf.find(name, "BF16", rows * cols, 2, &e));
+    LBK_TRY(dev_alloc(owner, rows * cols * 2, reinterpret_cast<void **>(out)));
+    return tf.sg.copy_linear(e->begin, rows * cols * 2, *out, name.c_str());
+}
+
+bool json_positive(const Json *j, size_t *out) {
+    if (!j || j->kind != Json::Num || j->num < 1 || j->num > 1e9 || j->num != std::floor(j->num)) return false;
+    *out = static_cast<size_t>(j->num);
+    return true;
 }
 
 // Continuous batching over one cache of `slots` sequences: what the reference's server would need in
@@ -193,10 +262,13 @@ int ensure_graph(Model *m, Cache *c) {
     Ctx *ctx = m->ctx;
     cudaStream_t st = ctx->own_stream;
     std::vector<int32_t> saved(c->b);
-    LBK_CUDA(cudaMemcpy(saved.data(), c->pos, c->b * 4, cudaMemcpyDeviceToHost));
-    LBK_TRY(enqueue_full_step(m, c, st));  // eager warm-up: writes the K/V rows of the saved positions, which the real step rewrites
+    LBK_CUDA(cudaMemcpy(saved.data(), c->active, c->b * 4, cudaMemcpyDeviceToHost));
+    // Eager warm-up with no sequence taking part: positions and recurrent states stay; cache rows written at the present
+    // positions are rewritten by the real step.
+    LBK_CUDA(cudaMemsetAsync(c->active, 0, c->b * 4, st));
+    LBK_TRY(enqueue_full_step(m, c, st));
+    LBK_CUDA(cudaMemcpyAsync(c->active, saved.data(), c->b * 4, cudaMemcpyHostToDevice, st));
     LBK_CUDA(cudaStreamSynchronize(st));
-    LBK_CUDA(cudaMemcpy(c->pos, saved.data(), c->b * 4, cudaMemcpyHostToDevice));
     const uint64_t before = ctx->launches;
     LBK_CUDA(cudaStreamBeginCapture(st, cudaStreamCaptureModeThreadLocal));
     const int status = enqueue_full_step(m, c, st);
@@ -384,6 +456,7 @@ int lbk_kv_cache_reset(lbk_kv_cache *cp) {
     LBK_CUDA(cudaSetDevice(c->model->ctx->device));
     LBK_CUDA(cudaDeviceSynchronize());
     LBK_CUDA(cudaMemset(c->pos, 0, c->b * 4));
+    LBK_CUDA(cudaDeviceSynchronize());  // the context's own stream does not wait for the default one
     c->lens.assign(c->b, 0);
     return LBK_OK;
 }
@@ -437,6 +510,7 @@ int lbk_kv_cache_reset_seq(lbk_kv_cache *cp, size_t seq) {
     LBK_CUDA(cudaSetDevice(c->model->ctx->device));
     LBK_CUDA(cudaDeviceSynchronize());
     LBK_CUDA(cudaMemset(c->pos + seq, 0, 4));
+    LBK_CUDA(cudaDeviceSynchronize());
     c->lens[seq] = 0;
     return LBK_OK;
 }

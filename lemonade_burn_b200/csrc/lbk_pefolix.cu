@@ -35,8 +35,6 @@ struct PefolixLayer {
     DenseWeight eup, edown, sdown;  // experts stacked
 };
 
-size_t pad16(size_t v) { return (v + 15) / 16 * 16; }
-
 struct PefolixCache;
 
 struct PefolixModel : Model {
@@ -377,63 +375,6 @@ int PefolixModel::enqueue_head(const float *rows, size_t n, float *logits, cudaS
 }
 
 // ---- loading --------------------------------------------------------------------------------------
-struct Loader {
-    Ctx *ctx;
-    PefolixModel *m;
-    TensorFile &tf;
-
-    // rows and columns of a bf16 matrix
-    int shape(const std::string &name, size_t *rows, size_t *cols) const {
-        const auto it = tf.entries.find(name);
-        if (it == tf.entries.end()) return fail(LBK_ERR_INVALID, "%s: tensor %s is missing", tf.path.c_str(), name.c_str());
-        if (it->second.shape.size() != 2) return fail(LBK_ERR_SHAPE, "%s: %s is not a matrix", tf.path.c_str(), name.c_str());
-        *rows = it->second.shape[0];
-        *cols = it->second.shape[1];
-        return LBK_OK;
-    }
-    int vec(const std::string &name, size_t n, float **out) {
-        const TensorEntry *e;
-        LBK_TRY(tf.find(name, "BF16", n, 2, &e));
-        std::vector<uint16_t> raw(n);
-        if (pread(tf.sg.fd, raw.data(), n * 2, static_cast<off_t>(tf.sg.data0 + e->begin)) != static_cast<ssize_t>(n * 2))
-            return fail(LBK_ERR_INVALID, "cannot read %s", name.c_str());
-        std::vector<float> f(n);
-        for (size_t i = 0; i < n; ++i) {
-            const uint32_t bits = static_cast<uint32_t>(raw[i]) << 16;
-            memcpy(&f[i], &bits, 4);
-        }
-        LBK_TRY(dev_alloc(m->device_allocs, n * 4, reinterpret_cast<void **>(out)));
-        LBK_CUDA(cudaMemcpy(*out, f.data(), n * 4, cudaMemcpyHostToDevice));
-        tf.sg.bytes_read += n * 2;
-        tf.sg.bytes_to_device += n * 4;
-        return LBK_OK;
-    }
-    // matrices of the same width, one under the other
-    int stack(const std::vector<std::string> &names, const std::vector<size_t> &rows, size_t cols, DenseWeight *out) {
-        size_t total = 0;
-        for (size_t r : rows) total += r;
-        const size_t pitch = dense_pitch(cols);
-        uint16_t *dev = nullptr;
-        LBK_TRY(dev_alloc(m->device_allocs, total * pitch * 2, reinterpret_cast<void **>(&dev)));
-        if (pitch != cols) LBK_CUDA(cudaMemsetAsync(dev, 0, total * pitch * 2, ctx->own_stream));
-        size_t at = 0;
-        for (size_t i = 0; i < names.size(); ++i) {
-            const TensorEntry *e;
-            LBK_TRY(tf.find(names[i], "BF16", rows[i] * cols, 2, &e));
-            LBK_TRY(tf.sg.copy_rows(e->begin, rows[i], cols * 2, dev + at * pitch, pitch * 2, names[i].c_str()));
-            at += rows[i];
-        }
-        *out = DenseWeight{dev, total, cols, pitch};
-        return LBK_OK;
-    }
-};
-
-bool positive(const Json *j, size_t *out) {
-    if (!j || j->kind != Json::Num || j->num < 1 || j->num > 1e9 || j->num != std::floor(j->num)) return false;
-    *out = static_cast<size_t>(j->num);
-    return true;
-}
-
 int load_pefolix(Ctx *ctx, const std::string &dir, const Json &cj, int compute, int, int world, std::unique_ptr<Model> &out) {
     if (world > 1) return fail(LBK_ERR_UNSUPPORTED, "the Pefolix family is not sharded over ranks");
     PefolixModel *m = new PefolixModel();
@@ -446,25 +387,18 @@ int load_pefolix(Ctx *ctx, const std::string &dir, const Json &cj, int compute, 
     m->eps = static_cast<float>(eps->num);
     TensorFile tf;
     LBK_TRY(tf.open_file(dir + "/model.safetensors", ctx->own_stream));
-    Loader ld{ctx, m, tf};
+    WeightLoader ld{ctx, m->device_allocs, tf};
     size_t vocab = 0, width = 0, v2 = 0, w2 = 0;
     LBK_TRY(ld.shape("embed", &vocab, &width));
     LBK_TRY(ld.shape("head", &v2, &w2));
     size_t cv = 0, cw = 0;
-    if (!vocab || !width || v2 != vocab || w2 != width || (positive(cj.get("vocab"), &cv) && cv != vocab) || (positive(cj.get("width"), &cw) && cw != width))
+    if (!vocab || !width || v2 != vocab || w2 != width || (json_positive(cj.get("vocab"), &cv) && cv != vocab) || (json_positive(cj.get("width"), &cw) && cw != width))
         return fail(LBK_ERR_SHAPE, "%s: embed is [%zu, %zu], head [%zu, %zu]; config.json says vocab %zu, width %zu", tf.path.c_str(), vocab, width, v2, w2, cv, cw);
     m->width = width;
-    {
-        const TensorEntry *e;
-        LBK_TRY(tf.find("embed", "BF16", vocab * width, 2, &e));
-        LBK_TRY(dev_alloc(m->device_allocs, vocab * width * 2, reinterpret_cast<void **>(&m->embed)));
-        LBK_TRY(tf.sg.copy_linear(e->begin, vocab * width * 2, m->embed, "embed"));
-        uint16_t *hd = nullptr;
-        LBK_TRY(tf.find("head", "BF16", vocab * width, 2, &e));
-        LBK_TRY(dev_alloc(m->device_allocs, vocab * width * 2, reinterpret_cast<void **>(&hd)));
-        LBK_TRY(tf.sg.copy_linear(e->begin, vocab * width * 2, hd, "head"));
-        m->head = DenseWeight{hd, vocab, width, width};
-    }
+    uint16_t *hd = nullptr;
+    LBK_TRY(ld.table("embed", vocab, width, &m->embed));
+    LBK_TRY(ld.table("head", vocab, width, &hd));
+    m->head = DenseWeight{hd, vocab, width, width};
     LBK_TRY(ld.vec("final.norm", width, &m->final_norm));
     size_t first_ff = 0;
     for (size_t i = 0; i < layers->arr.size(); ++i) {
@@ -475,8 +409,8 @@ int load_pefolix(Ctx *ctx, const std::string &dir, const Json &cj, int compute, 
             return fail(LBK_ERR_UNSUPPORTED, "%s/config.json: layer %zu has no mixer this family knows (attention)", dir.c_str(), i);
         PefolixLayer l;
         const Json *scale = mx->get("scale");
-        if (!positive(mx->get("heads"), &l.heads) || !positive(mx->get("kv_heads"), &l.kv_heads) || !positive(mx->get("dim"), &l.dim) ||
-            !positive(mx->get("vdim"), &l.vdim) || l.heads % l.kv_heads || !scale || scale->kind != Json::Num)
+        if (!json_positive(mx->get("heads"), &l.heads) || !json_positive(mx->get("kv_heads"), &l.kv_heads) || !json_positive(mx->get("dim"), &l.dim) ||
+            !json_positive(mx->get("vdim"), &l.vdim) || l.heads % l.kv_heads || !scale || scale->kind != Json::Num)
             return fail(LBK_ERR_INVALID, "%s/config.json: layer %zu: heads, kv_heads, dim, vdim or scale is missing or inconsistent", dir.c_str(), i);
         if (l.dim > 512 || l.vdim > 512) return fail(LBK_ERR_UNSUPPORTED, "layer %zu: head sizes of at most 512", i);
         l.dimp = pad16(l.dim);
@@ -485,8 +419,8 @@ int load_pefolix(Ctx *ctx, const std::string &dir, const Json &cj, int compute, 
         const Json *mask = mx->get("mask");
         if (mask && mask->kind == Json::Obj) {
             size_t v = 0;
-            if (positive(mask->get("size"), &v)) l.mask.size = static_cast<int>(v);
-            if (positive(mask->get("keep_first"), &v)) l.mask.keep_first = static_cast<int>(v);
+            if (json_positive(mask->get("size"), &v)) l.mask.size = static_cast<int>(v);
+            if (json_positive(mask->get("keep_first"), &v)) l.mask.keep_first = static_cast<int>(v);
         }
         LBK_TRY(ld.vec(p + "norm1", width, &l.norm1));
         LBK_TRY(ld.vec(p + "norm1b", width, &l.norm1b));
@@ -507,7 +441,7 @@ int load_pefolix(Ctx *ctx, const std::string &dir, const Json &cj, int compute, 
             } else if (ks == "moe") {
                 l.kind = PefolixLayer::Moe;
                 const Json *router = mlp->get("router"), *shared = mlp->get("shared");
-                if (!router || !positive(router->get("experts"), &l.experts) || !positive(router->get("top"), &l.top) || l.top > l.experts)
+                if (!router || !json_positive(router->get("experts"), &l.experts) || !json_positive(router->get("top"), &l.top) || l.top > l.experts)
                     return fail(LBK_ERR_INVALID, "%s/config.json: layer %zu: mlp.router", dir.c_str(), i);
                 if (l.experts > 1024 || l.top > 32) return fail(LBK_ERR_UNSUPPORTED, "layer %zu: at most 1024 experts, 32 of them per token", i);
                 LBK_TRY(ld.shape(p + "mlp.e0.up", &l.ff, &cols));

@@ -1,5 +1,5 @@
-// What the model runtime (lbk_model.cu) and the model families (lbk_bitnet.cu, lbk_pefolix.cu) share: the JSON
-// reader, the safetensors file and its staged copies to the device, and the two base classes. A family
+// What the model runtime (lbk_model.cu) and the model families (lbk_bitnet.cu, lbk_pefolix.cu, lbk_dugulorn.cu) share:
+// the JSON reader, the safetensors file and its staged copies to the device, and the two base classes. A family
 // derives from Model and Cache, registers a loader under the architecture name its config.json carries, and
 // supplies the launches of a decode step and of a prompt pass; positions, slots, graphs, logits rows, greedy
 // tokens and the batcher are the runtime's.
@@ -20,6 +20,7 @@
 #include <string>
 #include <vector>
 
+#include "lbk_dense.cuh"
 #include "lbk_internal.cuh"
 
 namespace lbk {
@@ -319,6 +320,26 @@ inline size_t json_size(const Json *j, bool &ok) {
     }
     return static_cast<size_t>(j->num);
 }
+
+// ---- weights of a family from its tensor file (bf16 tensors) -----------------------------------------
+struct WeightLoader {
+    Ctx *ctx;
+    std::vector<void *> &owner;  // who frees the device memory
+    TensorFile &tf;
+
+    // rows and columns of a matrix
+    int shape(const std::string &name, size_t *rows, size_t *cols) const;
+    // a vector as f32, `add` added to every value
+    int vec(const std::string &name, size_t n, float **out, float add = 0.0f);
+    // numbers that are not in the file
+    int floats(const std::vector<float> &v, float **out);
+    // matrices of the same width, one under the other; an empty name stands for that many rows of zeros
+    int stack(const std::vector<std::string> &names, const std::vector<size_t> &rows, size_t cols, DenseWeight *out);
+    // a table [rows][cols], rows back to back
+    int table(const std::string &name, size_t rows, size_t cols, uint16_t **out);
+};
+// a whole number of at least 1
+bool json_positive(const Json *j, size_t *out);
 
 // ---- the base classes ---------------------------------------------------------------------------
 struct Model;

@@ -10,17 +10,14 @@ mix.q, mix.k, mix.v, mix.o, mlp.gate, up, down, or mlp.router, e<k>.up, e<k>.dow
 """
 from __future__ import annotations
 
-import json
-import struct
-from pathlib import Path
 from typing import Dict, Iterator, Optional, Tuple
 
 import numpy as np
 
+from .checkpoint import FILE_NAME, bf16_bits, bf16_values, save_checkpoint  # noqa: F401
 from .runtime import NativeModel, register
 
 ARCHITECTURE = "Pefolix"
-FILE_NAME = "model.safetensors"
 
 
 class NativePefolix(NativeModel):
@@ -83,16 +80,6 @@ def tensor_shapes(cfg: dict) -> Iterator[Tuple[str, Tuple[int, ...]]]:
     yield "head", (V, W)
 
 
-def bf16_bits(a: np.ndarray) -> np.ndarray:
-    """float32 -> bf16 bits, round to nearest even."""
-    u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
-    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
-
-
-def bf16_values(bits: np.ndarray) -> np.ndarray:
-    return (bits.astype(np.uint32) << 16).view(np.float32)
-
-
 def random_checkpoint(cfg: dict, seed: int = 0) -> Dict[str, np.ndarray]:
     """Random weights as bf16 bits: matrices N(0, 1 / columns), norm weights near 1, embedding N(0, 1)."""
     rng = np.random.default_rng(seed)
@@ -105,21 +92,3 @@ def random_checkpoint(cfg: dict, seed: int = 0) -> Dict[str, np.ndarray]:
             a *= shape[1] ** -0.5
         out[name] = bf16_bits(a)
     return out
-
-
-def save_checkpoint(directory, cfg: dict, tensors: Dict[str, np.ndarray]) -> None:
-    """config.json + model.safetensors; `tensors` are bf16 bits (uint16)."""
-    directory = Path(directory)
-    directory.mkdir(parents=True, exist_ok=True)
-    (directory / "config.json").write_text(json.dumps(cfg))
-    head, off = {}, 0
-    for name, t in tensors.items():
-        head[name] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [off, off + 2 * t.size]}
-        off += 2 * t.size
-    text = json.dumps(head).encode()
-    text += b" " * (-len(text) % 8)
-    with open(directory / FILE_NAME, "wb") as f:
-        f.write(struct.pack("<Q", len(text)))
-        f.write(text)
-        for t in tensors.values():
-            f.write(np.ascontiguousarray(t, dtype="<u2").tobytes())

@@ -35,7 +35,7 @@ def load_model(directory, ctx: Optional[Context] = None, dtype: str = "bfloat16"
     if arch == "" and arch not in _FAMILIES:
         from . import model  # noqa: F401  (registers BitNet; needs torch)
     elif arch not in _FAMILIES:
-        from . import pefolix  # noqa: F401
+        from . import dugulorn, pefolix  # noqa: F401
     if arch not in _FAMILIES:
         raise ValueError(f"no model family for architecture {arch!r} (known: {sorted(_FAMILIES)})")
     if arch == "":

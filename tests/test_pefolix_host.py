@@ -25,11 +25,13 @@ def test_registry_by_architecture(tmp_path):
 
 
 def test_build_parts_cover_the_sources():
-    """Every source is the runtime's or one family's, and a family's part does not name another's."""
+    """Every source is the runtime's or a family's; families may share kernel files, not each other's model file."""
     from lemonade_burn_b200 import build
     assert sorted(build.SOURCES) == sorted(p.name for p in build.CSRC.glob("*.cu"))
     assert len(build.SOURCES) == len(set(build.SOURCES))
-    assert set(build.FAMILIES) == {"", "Pefolix"}
+    assert set(build.FAMILIES) == {"", "Pefolix", "Dugulorn"}
+    for name, sources in build.FAMILIES.items():
+        assert not any(f"lbk_{other.lower()}.cu" in sources for other in build.FAMILIES if other and other != name)
     build.build()
     assert build.library_for("Pefolix") == build.LIB   # the whole library is there and fresh
 
