@@ -1070,14 +1070,18 @@ def main():
                     help="side measurements to add under `extra` (comma list of sustained, config0, config2, config3, convert, tp; "
                          "'none' for a profiler run)")
     ap.add_argument("--decode-batches", type=int, nargs="+", default=[1, 16], help="batch sizes of the config-3 decode step")
-    ap.add_argument("--workload", choices=["sweep", "pefolix"], default="sweep",
-                    help="sweep: the headline; pefolix: the Pefolix family beside BitNet at equal sizes (bench_pefolix.py, one GPU)")
-    ap.add_argument("--parts", default="kernels,models", help="with --workload pefolix: which parts to run")
+    ap.add_argument("--workload", choices=["sweep", "pefolix", "dugulorn"], default="sweep",
+                    help="sweep: the headline; pefolix: the Pefolix family beside BitNet at equal sizes (bench_pefolix.py, one GPU); "
+                         "dugulorn: the Dugulorn family beside Pefolix (bench_dugulorn.py, one GPU)")
+    ap.add_argument("--parts", default="kernels,models", help="with --workload pefolix or dugulorn: which parts to run")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     if args.workload == "pefolix":
         import bench_pefolix
         return bench_pefolix.run(args, ClockSampler)
+    if args.workload == "dugulorn":
+        import bench_dugulorn
+        return bench_dugulorn.run(args, ClockSampler)
     args.extras = set(args.extras.split(","))
     if args.impl == "reference":
         return run_reference(args)

@@ -395,7 +395,7 @@ int lbk_argmax(lbk_ctx *ctx, const float *logits_dev, size_t rows, size_t n, int
 int lbk_advance_pos(lbk_ctx *ctx, int32_t *pos_dev, void *stream);
 
 /* ---- bf16-weight layers (no counterpart in the reference, whose projections are ternary) ------------
- * The mechanisms of the Pefolix family, each callable alone. Row pitches are in values; rows of the compute
+ * The mechanisms of the Pefolix and Dugulorn families, each callable alone. Row pitches are in values; rows of the compute
  * type (LBK_COMPUTE_BF16: bf16 bits, LBK_COMPUTE_F32: float) that feed a projection have a pitch of a
  * multiple of 64 and hold numbers (no NaN) up to it.
  * lbk_sandwich_norm  x_dev f32 [rows][n]: with y_dev, x += layer_norm(y) * w_post; with w_dev, the rows
@@ -426,14 +426,82 @@ int lbk_attn_window(lbk_ctx *ctx, int compute, const void *q_dev, const void *kc
                     size_t n, int rows_of_seq, size_t heads, size_t kv_heads, size_t dim, size_t dim_pitch, size_t vdim, size_t vdim_pitch,
                     size_t cap, float scale, size_t window, size_t keep_first, int distance_bias, float *scratch_dev, void *out_dev,
                     size_t out_pitch, void *stream);
+/* The same with RMS norms, x / sqrt(mean(x^2) + eps). Without w_dev the outputs are the sum itself (both calls). */
+int lbk_sandwich_rms_norm(lbk_ctx *ctx, float *x_dev, const float *y_dev, const float *w_post_dev, const float *w_dev, size_t rows, size_t n,
+                          float eps, float *out_f32_dev, uint16_t *out_bf16_dev, size_t out_bf16_pitch, void *stream);
+/* A projection with a bias (f32, may be null) and an activation (LBK_ACT_*) on the output rows below act_rows; with
+ * out_f32 the values as they are. */
+#define LBK_ACT_NONE 0
+#define LBK_ACT_RELU2 1
+#define LBK_ACT_SILU 2
+int lbk_dense_linear_act(lbk_ctx *ctx, int compute, const void *x_dev, size_t x_pitch, size_t m, const uint16_t *w_dev, size_t w_pitch,
+                         size_t w_rows, size_t cols, const float *bias_dev, int act, size_t act_rows, void *out_dev, size_t out_pitch,
+                         int out_f32, void *stream);
+
+/* Latent attention: a position caches a row of lbk_latent_pitch values, the latent (kv_rank values) and, from
+ * lbk_latent_key_at on, a rotated key part that all heads share; zeros between. Rotation turns neighbouring dimensions
+ * (2i, 2i + 1) by position * freq[i], cos and sin times rot_factor; lbk_rotation_frequencies fills freq (host) with
+ * base^(-2i / dims), or with `yarn` = {factor, original, fast, slow} the interpolated ones and the factor.
+ * lbk_latent_prep   z f32 [rows][z_pitch] = [query latent q_rank | latent kv_rank | key part rot_dim | ...]: the normed
+ *                   query latent to cq; with cache_dev the normed latent and rotated key part into the rows' places
+ *                   (without, z has no latent and key part).
+ * lbk_latent_attn   q [rows][heads][lbk_latent_query_pitch], unrotated part first, the part to rotate from
+ *                   lbk_latent_query_rot_at on (q may be changed); ukv: keys' [heads * dim][kv_rank], then values'
+ *                   [heads * vdim][kv_rank] weights. out [rows][heads * vdim] = softmax((q . k) * scale) v times
+ *                   sigmoid(gate[row * gate_pitch + head]). length 0: the absorbing form; length > 0 (bf16, prompt rows,
+ *                   lbk_latent_expand_supported): keys and values of that many positions are written out first. work:
+ *                   lbk_latent_work_bytes. rows_of_seq and pos_dev as in lbk_attn_window. */
+typedef struct lbk_latent_desc {
+    size_t heads, dim, rot_dim, vdim, kv_rank, q_rank;
+    const double *freq_dev; /* [rot_dim / 2] */
+    float rot_factor;
+} lbk_latent_desc;
+size_t lbk_latent_pitch(const lbk_latent_desc *desc);
+size_t lbk_latent_key_at(const lbk_latent_desc *desc);
+size_t lbk_latent_query_pitch(const lbk_latent_desc *desc);
+size_t lbk_latent_query_rot_at(const lbk_latent_desc *desc);
+int lbk_latent_expand_supported(const lbk_latent_desc *desc);
+int lbk_rotation_frequencies(size_t dims, double base, const double *yarn, double *freq_out, float *factor_out);
+int lbk_latent_prep(lbk_ctx *ctx, int compute, const lbk_latent_desc *desc, const float *z_dev, size_t z_pitch, size_t rows, int rows_of_seq,
+                    const int32_t *pos_dev, size_t cap, const float *q_norm_dev, const float *kv_norm_dev, float eps, void *cq_dev,
+                    size_t cq_pitch, void *cache_dev, void *stream);
+size_t lbk_latent_work_bytes(lbk_ctx *ctx, int compute, const lbk_latent_desc *desc, size_t rows, size_t cap, size_t length);
+int lbk_latent_attn(lbk_ctx *ctx, int compute, const lbk_latent_desc *desc, void *q_dev, size_t rows, int rows_of_seq, const int32_t *pos_dev,
+                    size_t cap, const void *cache_dev, const uint16_t *ukv_dev, size_t ukv_pitch, float scale, const float *gate_dev,
+                    size_t gate_pitch, size_t length, void *work_dev, void *out_dev, size_t out_pitch, void *stream);
+
+/* Linear recurrences over a state S [dim x vdim] per head and sequence, f32, zero in front of position 0:
+ *   plain  S <- decay_h S + k v^T;  o = S^T q         x rows hold q, k, v [heads x dim, heads x dim, heads x vdim]
+ *   delta  S <- g S (per key channel); u = beta (v - S^T k); S <- S + k u^T;  o = S^T q
+ *          x rows hold q, k [kv_heads x dim], v [heads x vdim]; each channel passes a causal convolution of `taps`
+ *          inputs (conv f32 [taps][channels], the last row meets the token itself) and silu; q and k become unit
+ *          vectors, x / sqrt(sum x^2 + 1e-6), q times dim^-1/2; g = exp(-exp(a_log[h]) softplus(a + dt_bias)) with a
+ *          [rows][heads * dim]; beta = sigmoid(b [rows][heads]).
+ * state [seq][lbk_recurrence_state_floats], ring [seq][taps][channels] of the compute type (delta), o [rows][heads * vdim].
+ * records (rows_of_seq >= 0): lbk_recurrence_record_floats(record_rows). active_dev (may be null): sequences with 0 keep
+ * their state (rows_of_seq = -1).
+ * lbk_gated_norm: out = o / sqrt(mean over its group of `group` values + eps) * w[place in the group] * sigmoid(gate). */
+typedef struct lbk_recurrence_desc {
+    int delta;
+    size_t heads, kv_heads, dim, vdim, taps;
+} lbk_recurrence_desc;
+size_t lbk_recurrence_state_floats(const lbk_recurrence_desc *desc);
+size_t lbk_recurrence_record_floats(const lbk_recurrence_desc *desc, size_t rows);
+int lbk_recurrence(lbk_ctx *ctx, int compute, const lbk_recurrence_desc *desc, const void *x_dev, size_t x_pitch, size_t rows, int rows_of_seq,
+                   const int32_t *pos_dev, const int32_t *active_dev, size_t cap, const float *decay_dev, const float *conv_dev,
+                   void *ring_dev, const float *a_dev, const float *a_log_dev, const float *dt_bias_dev, const float *b_dev,
+                   float *state_dev, float *records_dev, size_t record_rows, float *o_dev, void *stream);
+int lbk_gated_norm(lbk_ctx *ctx, int compute, const float *o_dev, size_t rows, size_t n, size_t group, const float *w_dev,
+                   const void *gate_dev, size_t gate_pitch, float eps, void *out_dev, size_t out_pitch, void *stream);
 size_t lbk_moe_route_ints(size_t n, size_t experts, size_t top);
 int lbk_moe_route(lbk_ctx *ctx, const float *z_dev, size_t z_pitch, size_t n, size_t experts, size_t top, int32_t *scratch_dev,
                   const uint16_t *x_dev, size_t x_pitch, uint16_t *sorted_dev, int32_t *ids_out_dev, float *weights_out_dev,
                   int32_t *place_out_dev, int32_t *offs_out_dev, void *stream);
 
 /* ---- the decoder as a native runtime (crates/lb-model/src/model.rs) ----------------------------
- * Two families: BitNet (below) and Pefolix (`dir/config.json` with "architecture": "Pefolix" and
- * `dir/model.safetensors`, bf16 tensors), which has the same calls.
+ * Three families: BitNet (below), Pefolix and Dugulorn (`dir/config.json` with "architecture": "Pefolix" or
+ * "Dugulorn" and `dir/model.safetensors`, bf16 tensors), which have the same calls. A Dugulorn cache holds latents
+ * and recurrent states in the place of keys and values.
  * lbk_model_load      BitNet::load (model.rs:149-232): `dir/config.json` + `dir/model.lbt.safetensors`
  *                     as lb-convert writes them; the format check and the supported family
  *                     (relu2, tied embeddings) are the reference's; head_dim must be 128.

@@ -92,6 +92,21 @@ SYMBOLS = [
     ("lbk_tp_gather_f32", _vp, [_vp]),
     ("lbk_tp_argmax", _i, [_vp, _vp, _vp, _sz, _sz, _vp, _vp]),
     ("lbk_sandwich_norm", _i, [_vp, _vp, _vp, _vp, _vp, _sz, _sz, _f, _vp, _vp, _sz, _vp]),
+    ("lbk_sandwich_rms_norm", _i, [_vp, _vp, _vp, _vp, _vp, _sz, _sz, _f, _vp, _vp, _sz, _vp]),
+    ("lbk_dense_linear_act", _i, [_vp, _i, _vp, _sz, _sz, _vp, _sz, _sz, _sz, _vp, _i, _sz, _vp, _sz, _i, _vp]),
+    ("lbk_latent_pitch", _sz, [_vp]),
+    ("lbk_latent_key_at", _sz, [_vp]),
+    ("lbk_latent_query_pitch", _sz, [_vp]),
+    ("lbk_latent_query_rot_at", _sz, [_vp]),
+    ("lbk_latent_expand_supported", _i, [_vp]),
+    ("lbk_rotation_frequencies", _i, [_sz, C.c_double, _vp, _vp, _vp]),
+    ("lbk_latent_prep", _i, [_vp, _i, _vp, _vp, _sz, _sz, _i, _vp, _sz, _vp, _vp, _f, _vp, _sz, _vp, _vp]),
+    ("lbk_latent_work_bytes", _sz, [_vp, _i, _vp, _sz, _sz, _sz]),
+    ("lbk_latent_attn", _i, [_vp, _i, _vp, _vp, _sz, _i, _vp, _sz, _vp, _vp, _sz, _f, _vp, _sz, _sz, _vp, _vp, _sz, _vp]),
+    ("lbk_recurrence_state_floats", _sz, [_vp]),
+    ("lbk_recurrence_record_floats", _sz, [_vp, _sz]),
+    ("lbk_recurrence", _i, [_vp, _i, _vp, _vp, _sz, _sz, _i, _vp, _vp, _sz, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp, _vp]),
+    ("lbk_gated_norm", _i, [_vp, _i, _vp, _sz, _sz, _sz, _vp, _vp, _sz, _f, _vp, _sz, _vp]),
     ("lbk_dense_linear", _i, [_vp, _i, _vp, _sz, _sz, _vp, _sz, _sz, _sz, _i, _sz, _i, _vp, _sz, _i, _vp, _sz, _vp]),
     ("lbk_attn_window_scratch", _sz, [_sz, _sz, _sz]),
     ("lbk_attn_window", _i, [_vp, _i, _vp, _vp, _vp, _vp, _sz, _i, _sz, _sz, _sz, _sz, _sz, _sz, _sz, _f, _sz, _sz, _i, _vp, _vp, _sz, _vp]),

@@ -947,3 +947,28 @@ extern "C" int lbk_dense_linear(lbk_ctx *c, int compute, const void *x_dev, size
     d.offs = expert_offs_dev;
     return launch_dense(ctx, d, static_cast<cudaStream_t>(stream));
 }
+
+extern "C" int lbk_dense_linear_act(lbk_ctx *c, int compute, const void *x_dev, size_t x_pitch, size_t m, const uint16_t *w_dev, size_t w_pitch,
+                                    size_t w_rows, size_t cols, const float *bias_dev, int act, size_t act_rows, void *out_dev, size_t out_pitch,
+                                    int out_f32, void *stream) {
+    if (!c) return fail(LBK_ERR_INVALID, "lbk_dense_linear_act: context is null");
+    Ctx *ctx = reinterpret_cast<Ctx *>(c);
+    if (m && (!x_dev || !w_dev || !out_dev)) return fail(LBK_ERR_INVALID, "lbk_dense_linear_act: null buffer");
+    if (w_pitch % 64 || w_pitch < cols || x_pitch < w_pitch || x_pitch % 64) return fail(LBK_ERR_SHAPE, "lbk_dense_linear_act: pitches are multiples of 64 columns that cover the row");
+    if (act != kActNone && act != kActRelu2 && act != kActSilu) return fail(LBK_ERR_INVALID, "lbk_dense_linear_act: unknown activation %d", act);
+    LBK_CUDA(cudaSetDevice(ctx->device));
+    DenseCall d;
+    d.compute = compute;
+    d.x = x_dev;
+    d.ldx = static_cast<long>(x_pitch);
+    d.m = m;
+    d.w = DenseWeight{w_dev, w_rows, cols, w_pitch};
+    d.out_rows = w_rows;
+    d.epi.kind = out_f32 ? kEpiF32 : kEpiElem;
+    d.epi.act = act;
+    if (act_rows < w_rows) d.epi.act_rows = static_cast<int>(act_rows);
+    d.epi.bias = bias_dev;
+    d.epi.out = out_dev;
+    d.epi.ld = static_cast<long>(out_pitch);
+    return launch_dense(ctx, d, static_cast<cudaStream_t>(stream));
+}

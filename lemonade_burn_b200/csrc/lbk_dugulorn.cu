@@ -15,9 +15,9 @@
 //
 // Launches of a decode step in bf16, after the sum and norm that the first projection of a sublayer does itself at one
 // or two sequences: latent attention [query latent, latent, key part, gates], norms + rotation + cache, queries, absorb,
-// attention, merge + values + gate, o; lightning [q, k, v, gate + silu], records, state, gated norm, o; delta rule
-// [q, k, v, both low ranks, beta], both second halves, records, state, gated norm, o; feed-forward up + bias + relu^2,
-// down + bias. A prompt pass runs the same calls on its rows, with latent attention in its expanding form.
+// attention, merge + values + gate, o; lightning [q, k, v, gate + silu], state, gated norm, o; delta rule [q, k, v,
+// both low ranks, beta], everything up to the gated norm, o; feed-forward up + bias + relu^2, down + bias. A prompt pass
+// has latent attention in its expanding form and takes the recurrences eight tokens at a time.
 #include "lbk_mixers.cuh"
 #include "lbk_runtime.cuh"
 
@@ -151,7 +151,7 @@ int DugulornModel::make_work(std::vector<void *> &owner, Work &w, size_t rows, b
     // rows of the absorbing form: all of them, or the short passes only
     const size_t few = !batch && expands(rows) ? std::min(rows, kExpandRows - 1) : rows;
     size_t in = 0, mid = 0, h = 0, z = 0, cq = 0, q = 0, ql = 0, gate = 0, a = 0, o = 0, records = 0, scratch = 0;
-    w.record_rows = std::min((rows + 3) / 4 * 4, kRecordRows);
+    w.record_rows = std::min((rows + 7) / 8 * 8, kRecordRows);
     for (const DugulornLayer &l : layers) {
         mid = std::max(mid, dense_pitch(l.out_width()));
         h = std::max(h, dense_pitch(l.ff));
@@ -165,8 +165,8 @@ int DugulornModel::make_work(std::vector<void *> &owner, Work &w, size_t rows, b
             in = std::max(in, dense_pitch(l.in.rows));
             z = std::max(z, l.heads);
             o = std::max(o, l.heads * l.vdim);
-            records = std::max(records, recur_record_floats(l.type == Mixer::Delta, batch ? rows : w.record_rows, batch, l.heads, l.dim, l.vdim));
-            if (l.type == Mixer::Delta) {
+            if (!batch) records = std::max(records, recur_record_floats(l.type == Mixer::Delta, w.record_rows, l.heads, l.dim, l.vdim));
+            if (l.type == Mixer::Delta && !batch) {
                 a = std::max(a, l.heads * l.dim);
                 gate = std::max(gate, dense_pitch(l.heads * l.vdim));
             }
@@ -292,8 +292,18 @@ int DugulornModel::enqueue_recurrent(const Pass &p, const DugulornLayer &l, size
     const bool delta = l.type == Mixer::Delta;
     const long ldin = static_cast<long>(dense_pitch(l.in.rows));
     const size_t hv = l.heads * l.vdim, qk = l.kv_heads * l.dim;
+    RecurCall r;
     GatedNormCall g;
-    if (delta) {
+    if (delta && p.seq < 0) {
+        r.a2 = l.a2;
+        r.g2 = l.g2;
+        r.a_at = static_cast<int>(l.a_at);
+        r.g_at = static_cast<int>(l.g_at);
+        r.norm_w = l.mix_norm;
+        r.eps = eps;
+        r.out = w.mid;
+        r.ldo = static_cast<long>(l.o.pitch);
+    } else if (delta) {
         DenseCall d;
         d.compute = compute;
         d.m = p.m;
@@ -320,7 +330,6 @@ int DugulornModel::enqueue_recurrent(const Pass &p, const DugulornLayer &l, size
         g.ldg = ldin;
         g.group = hv;
     }
-    RecurCall r;
     r.compute = compute;
     r.delta = delta;
     r.heads = l.heads;
@@ -352,6 +361,7 @@ int DugulornModel::enqueue_recurrent(const Pass &p, const DugulornLayer &l, size
     r.record_rows = w.record_rows;
     r.o = w.o;
     LBK_TRY(launch_recurrence(ctx, r, p.st));
+    if (r.out) return LBK_OK;
     g.compute = compute;
     g.o = w.o;
     g.rows = p.m;
@@ -624,15 +634,17 @@ struct LayerReader {
                          {qk, qk, hv, l.a_at - ch, ra, l.g_at - l.a_at - ra, rg, l.b_at - l.g_at - rg, l.heads}, m->width, &l.in));
         LBK_TRY(ld.stack({p + "mix.a2"}, {l.heads * l.dim}, ra, &l.a2));
         LBK_TRY(ld.stack({p + "mix.g2"}, {hv}, rg, &l.g2));
-        float *part[3] = {};
-        const size_t n[3] = {qk * l.taps, qk * l.taps, hv * l.taps};
-        const char *name[3] = {"mix.q.conv", "mix.k.conv", "mix.v.conv"};
-        LBK_TRY(dev_alloc(m->device_allocs, ch * l.taps * 4, reinterpret_cast<void **>(&l.conv)));
+        // [channels][taps] in the file, [taps][channels] on the device
+        std::vector<float> conv(ch * l.taps), part;
         size_t at = 0;
-        for (int k = 0; k < 3; at += n[k], ++k) {
-            LBK_TRY(ld.vec(p + name[k], n[k], &part[k]));
-            LBK_CUDA(cudaMemcpy(l.conv + at, part[k], n[k] * 4, cudaMemcpyDeviceToDevice));
+        const struct { const char *name; size_t n; } parts[3] = {{"mix.q.conv", qk}, {"mix.k.conv", qk}, {"mix.v.conv", hv}};
+        for (const auto &c : parts) {
+            LBK_TRY(ld.read(p + c.name, c.n * l.taps, part));
+            for (size_t k = 0; k < c.n; ++k)
+                for (size_t j = 0; j < l.taps; ++j) conv[j * ch + at + k] = part[k * l.taps + j];
+            at += c.n;
         }
+        LBK_TRY(ld.floats(conv, &l.conv));
         LBK_TRY(ld.vec(p + "mix.A_log", l.heads, &l.a_log));
         LBK_TRY(ld.vec(p + "mix.dt_bias", l.heads * l.dim, &l.dt_bias));
         return ld.vec(p + "mix.norm", l.vdim, &l.mix_norm);

@@ -13,7 +13,7 @@
 // projection as it lies there. Kernels:
 //
 //   latent_prep_kernel    a token's projections: norm of the query latent; norm of c and rotation of the key part, stored
-//                         into the cache. Angles: position * frequency in double, reduced to one turn, then sincosf.
+//                         into the cache. Angles: position * frequency in double, reduced to one turn, then sincospif.
 //   latent_rotate_kernel  rotated parts of all heads of the queries in place (expanding form)
 //   latent_absorb_kernel  W_uk,h^T q and the rotated part: a query against cache rows
 //   latent_attn_kernel    bf16: 16 or 32 heads x 64 positions at a time on mma.sync, the positions' rows staged once by
@@ -38,11 +38,10 @@ struct Angles {
 };
 // (cos, sin) of pair i at position pos
 __device__ __forceinline__ float2 turn(const Angles &r, int i, int pos) {
-    constexpr double kTurn = 6.283185307179586476925286766559;
-    double a = static_cast<double>(pos) * r.freq[i];
-    a -= kTurn * floor(a / kTurn);
+    constexpr double kPerTurn = 0.15915494309189533576888376337251;  // 1 / (2 pi)
+    const double a = static_cast<double>(pos) * r.freq[i] * kPerTurn;
     float s, c;
-    sincosf(static_cast<float>(a), &s, &c);
+    sincospif(2.0f * static_cast<float>(a - floor(a)), &s, &c);
     return make_float2(c * r.factor, s * r.factor);
 }
 Angles angles(const Rotation &r) { return Angles{r.freq, r.dims, r.factor}; }
@@ -63,22 +62,49 @@ template <typename T>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const PrepParams p) {
     ptx::pdl_trigger();
     ptx::pdl_wait();
-    __shared__ float s_red[32];
+    __shared__ float2 s_red[8];
     const int row = blockIdx.x, tid = threadIdx.x;
     const float *z = p.z + static_cast<size_t>(row) * p.ldz, *kv = z + p.q_rank;
+    constexpr int kHeld = 8;                               // the first values of a thread stay in registers
+    float held[kHeld];
     float sq = 0.0f, sk = 0.0f;
-    for (int i = tid; i < p.q_rank; i += 256) sq = fmaf(z[i], z[i], sq);
-    const float rq = 1.0f / sqrtf(dense::block_sum<256>(sq, s_red) / static_cast<float>(p.q_rank) + p.eps);
+#pragma unroll
+    for (int j = 0; j < kHeld; ++j) {
+        const int i = tid + 256 * j;
+        held[j] = i < p.q_rank ? z[i] : 0.0f;
+        sq = fmaf(held[j], held[j], sq);
+    }
+    for (int i = tid + 256 * kHeld; i < p.q_rank; i += 256) sq = fmaf(z[i], z[i], sq);
+    if (p.cache)
+        for (int i = tid; i < p.kv_rank; i += 256) sk = fmaf(kv[i], kv[i], sk);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+    }
+    if ((tid & 31) == 0) s_red[tid >> 5] = make_float2(sq, sk);
+    __syncthreads();
+    sq = sk = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+        sq += s_red[w].x;
+        sk += s_red[w].y;
+    }
+    const float rq = 1.0f / sqrtf(sq / static_cast<float>(p.q_rank) + p.eps);
     T *cq = static_cast<T *>(p.cq) + static_cast<size_t>(row) * p.ldq;
-    for (int i = tid; i < p.q_rank; i += 256) dense::put(cq + i, z[i] * rq * p.q_norm[i]);
+#pragma unroll
+    for (int j = 0; j < kHeld; ++j) {
+        const int i = tid + 256 * j;
+        if (i < p.q_rank) dense::put(cq + i, held[j] * rq * p.q_norm[i]);
+    }
+    for (int i = tid + 256 * kHeld; i < p.q_rank; i += 256) dense::put(cq + i, z[i] * rq * p.q_norm[i]);
     if (!p.cache) return;
     const int seq = p.rows_of_seq >= 0 ? p.rows_of_seq : row, pos = p.rows_of_seq >= 0 ? p.pos[0] + row : p.pos[row];
     if (pos < 0 || pos >= p.cap) {
         if (tid == 0) atomicExch(p.err_word, 7);
         return;
     }
-    for (int i = tid; i < p.kv_rank; i += 256) sk = fmaf(kv[i], kv[i], sk);
-    const float rk = 1.0f / sqrtf(dense::block_sum<256>(sk, s_red) / static_cast<float>(p.kv_rank) + p.eps);
+    const float rk = 1.0f / sqrtf(sk / static_cast<float>(p.kv_rank) + p.eps);
     T *dst = static_cast<T *>(p.cache) + (static_cast<size_t>(seq) * p.cap + pos) * p.pitch;
     for (int i = tid; i < p.kv_rank; i += 256) dense::put(dst + i, kv[i] * rk * p.kv_norm[i]);
     for (int i = tid; i < p.rot_dim / 2; i += 256) {
@@ -424,6 +450,7 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const OutParams p) {
     ptx::pdl_trigger();
     ptx::pdl_wait();
     extern __shared__ float s_dyn[];                         // [kOutTok][uv_pitch], [splits] weights
+    __shared__ float4 s_half[128];                           // the second half of the slices' sum (latents of up to 512)
     float *s_w = s_dyn + kOutTok * p.uv_pitch;
     const int h = blockIdx.x, e0 = blockIdx.y * kOutRows, t0 = blockIdx.z * kOutTok, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int toks = min(kOutTok, p.rows - t0);
@@ -456,13 +483,22 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const OutParams p) {
         for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
         __syncthreads();
         const float inv = 1.0f / sum;
-        for (int i = tid; i < p.uv_pitch; i += 256) {
-            float a = 0.0f;
-            if (i < p.kv_rank) {
-#pragma unroll 8
-                for (int s = 0; s < p.splits; ++s) a += s_w[s] * part[static_cast<size_t>(s) * prow + i];
+        // four values a thread, every second slice; what lies between kv_rank and kvp is zero
+        const int i = (tid & 127) * 4, half = tid >> 7;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < p.kvp) {
+#pragma unroll 16
+            for (int s = half; s < p.splits; s += 2) {
+                const float4 v = *reinterpret_cast<const float4 *>(part + static_cast<size_t>(s) * prow + i);
+                const float w = s_w[s];
+                a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
             }
-            x[i] = a * inv;
+        }
+        if (half) s_half[tid & 127] = a;
+        __syncthreads();
+        if (!half && i < p.uv_pitch) {
+            const float4 b = s_half[tid];
+            *reinterpret_cast<float4 *>(x + i) = make_float4((a.x + b.x) * inv, (a.y + b.y) * inv, (a.z + b.z) * inv, (a.w + b.w) * inv);
         }
     }
     __syncthreads();
@@ -731,3 +767,145 @@ int launch_latent_expanded(Ctx *ctx, const LatentAttnCall &c, cudaStream_t st) {
 }
 
 }  // namespace lbk
+
+using namespace lbk;
+
+namespace {
+
+LatentShape shape_of(const lbk_latent_desc &d) {
+    LatentShape s;
+    s.heads = d.heads;
+    s.dim = d.dim;
+    s.rot_dim = d.rot_dim;
+    s.vdim = d.vdim;
+    s.kv_rank = d.kv_rank;
+    s.q_rank = d.q_rank;
+    return s;
+}
+Rotation rotation_of(const lbk_latent_desc &d) {
+    Rotation r;
+    r.freq = d.freq_dev;
+    r.dims = static_cast<int>(d.rot_dim);
+    r.factor = d.rot_factor;
+    return r;
+}
+// parts of the work memory of one call, in 256-byte steps
+struct LatentWork {
+    size_t ql = 0, scratch = 0, ek = 0, ev = 0, zero = 0, total = 0, ecap = 0;
+    LatentWork(const Ctx *ctx, int compute, const LatentShape &s, size_t rows, size_t cap, size_t length) {
+        const size_t es = compute == LBK_COMPUTE_F32 ? 4 : 2;
+        auto take = [&](size_t bytes) {
+            const size_t at = total;
+            total += (bytes + 255) / 256 * 256;
+            return at;
+        };
+        if (length) {
+            ecap = length;
+            ek = take(s.heads * length * s.dp() * 2);
+            ev = take(s.heads * length * s.vp() * 2);
+            zero = take(4);
+        } else {
+            ql = take(rows * s.heads * s.pitch() * es);
+            scratch = take(latent_scratch(ctx, rows, s, compute == LBK_COMPUTE_F32 ? 1 : latent_splits(cap)) * 4);
+        }
+    }
+};
+
+}  // namespace
+
+extern "C" {
+
+size_t lbk_latent_pitch(const lbk_latent_desc *d) { return d ? shape_of(*d).pitch() : 0; }
+size_t lbk_latent_key_at(const lbk_latent_desc *d) { return d ? shape_of(*d).kvp() : 0; }
+size_t lbk_latent_query_pitch(const lbk_latent_desc *d) { return d ? shape_of(*d).qp() : 0; }
+size_t lbk_latent_query_rot_at(const lbk_latent_desc *d) { return d ? shape_of(*d).dp() : 0; }
+int lbk_latent_expand_supported(const lbk_latent_desc *d) { return d && latent_expand_supported(shape_of(*d)) ? 1 : 0; }
+
+int lbk_rotation_frequencies(size_t dims, double base, const double *yarn, double *freq_out, float *factor_out) {
+    if (!freq_out || !factor_out || dims == 0 || dims % 2 || base <= 0.0) return fail(LBK_ERR_INVALID, "lbk_rotation_frequencies: an even number of dimensions and a positive base");
+    YarnScaling y;
+    if (yarn) {
+        y.on = true;
+        y.factor = yarn[0];
+        y.original = yarn[1];
+        y.fast = yarn[2];
+        y.slow = yarn[3];
+    }
+    rotation_frequencies(dims, base, y, freq_out, factor_out);
+    return LBK_OK;
+}
+
+int lbk_latent_prep(lbk_ctx *c, int compute, const lbk_latent_desc *d, const float *z_dev, size_t z_pitch, size_t rows, int rows_of_seq,
+                    const int32_t *pos_dev, size_t cap, const float *q_norm_dev, const float *kv_norm_dev, float eps, void *cq_dev, size_t cq_pitch,
+                    void *cache_dev, void *stream) {
+    if (!c || !d) return fail(LBK_ERR_INVALID, "lbk_latent_prep: null argument");
+    Ctx *ctx = reinterpret_cast<Ctx *>(c);
+    LBK_CUDA(cudaSetDevice(ctx->device));
+    LatentPrepCall p;
+    p.compute = compute;
+    p.s = shape_of(*d);
+    p.z = z_dev;
+    p.ldz = static_cast<long>(z_pitch);
+    p.rows = rows;
+    p.rows_of_seq = rows_of_seq;
+    p.pos = pos_dev;
+    p.cap = cap;
+    p.q_norm = q_norm_dev;
+    p.kv_norm = kv_norm_dev;
+    p.eps = eps;
+    p.rot = rotation_of(*d);
+    p.cq = cq_dev;
+    p.ldq = static_cast<long>(cq_pitch);
+    p.cache = cache_dev;
+    return launch_latent_prep(ctx, p, static_cast<cudaStream_t>(stream));
+}
+
+size_t lbk_latent_work_bytes(lbk_ctx *c, int compute, const lbk_latent_desc *d, size_t rows, size_t cap, size_t length) {
+    return c && d ? LatentWork(reinterpret_cast<Ctx *>(c), compute, shape_of(*d), rows, cap, length).total : 0;
+}
+
+int lbk_latent_attn(lbk_ctx *c, int compute, const lbk_latent_desc *d, void *q_dev, size_t rows, int rows_of_seq, const int32_t *pos_dev, size_t cap,
+                    const void *cache_dev, const uint16_t *ukv_dev, size_t ukv_pitch, float scale, const float *gate_dev, size_t gate_pitch, size_t length,
+                    void *work_dev, void *out_dev, size_t out_pitch, void *stream) {
+    if (!c || !d || !work_dev) return fail(LBK_ERR_INVALID, "lbk_latent_attn: null argument");
+    if (ukv_pitch != dense_pitch(d->kv_rank)) return fail(LBK_ERR_SHAPE, "lbk_latent_attn: the weights' pitch is kv_rank rounded up to 64");
+    Ctx *ctx = reinterpret_cast<Ctx *>(c);
+    LBK_CUDA(cudaSetDevice(ctx->device));
+    LatentAttnCall a;
+    a.compute = compute;
+    a.s = shape_of(*d);
+    a.q = q_dev;
+    a.rows = rows;
+    a.rows_of_seq = rows_of_seq;
+    a.pos = pos_dev;
+    a.cap = cap;
+    a.cache = cache_dev;
+    const size_t kr = d->heads * d->dim, vr = d->heads * d->vdim;
+    a.ukv = DenseWeight{ukv_dev, kr + vr, d->kv_rank, ukv_pitch};
+    a.uk = DenseWeight{ukv_dev, kr, d->kv_rank, ukv_pitch};
+    a.uv = DenseWeight{ukv_dev + kr * ukv_pitch, vr, d->kv_rank, ukv_pitch};
+    a.scale = scale;
+    a.rot = rotation_of(*d);
+    a.gate = gate_dev;
+    a.ldg = static_cast<long>(gate_pitch);
+    a.out = out_dev;
+    a.ldo = static_cast<long>(out_pitch);
+    const LatentWork w(ctx, compute, a.s, rows, cap, length);
+    char *base = static_cast<char *>(work_dev);
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (length) {
+        a.length = length;
+        a.ek = base + w.ek;
+        a.ev = base + w.ev;
+        a.ecap = w.ecap;
+        a.zero = reinterpret_cast<int *>(base + w.zero);
+        LBK_CUDA(cudaMemsetAsync(base, 0, w.total, st));  // the padding of keys and values has to hold numbers
+        return launch_latent_expanded(ctx, a, st);
+    }
+    a.ql = base + w.ql;
+    a.scratch = reinterpret_cast<float *>(base + w.scratch);
+    a.splits = latent_splits(cap);
+    return launch_latent_absorbed(ctx, a, st);
+}
+
+}  // extern "C"

@@ -289,12 +289,13 @@ int launch_sandwich_norm(Ctx *ctx, const NormCall &c, cudaStream_t st) {
 
 using namespace lbk;
 
-extern "C" int lbk_sandwich_norm(lbk_ctx *c, float *x_dev, const float *y_dev, const float *w_post_dev, const float *w_dev, size_t rows, size_t n,
-                                 float eps, float *out_f32_dev, uint16_t *out_bf16_dev, size_t out_bf16_pitch, void *stream) {
-    if (!c) return fail(LBK_ERR_INVALID, "lbk_sandwich_norm: context is null");
+static int sandwich_norm(lbk_ctx *c, bool rms, float *x_dev, const float *y_dev, const float *w_post_dev, const float *w_dev, size_t rows, size_t n,
+                         float eps, float *out_f32_dev, uint16_t *out_bf16_dev, size_t out_bf16_pitch, void *stream) {
+    if (!c) return fail(LBK_ERR_INVALID, "sandwich norm: context is null");
     Ctx *ctx = reinterpret_cast<Ctx *>(c);
     LBK_CUDA(cudaSetDevice(ctx->device));
     NormCall k;
+    k.rms = rms;
     k.x = x_dev;
     k.y = y_dev;
     k.w_post = w_post_dev;
@@ -306,4 +307,14 @@ extern "C" int lbk_sandwich_norm(lbk_ctx *c, float *x_dev, const float *y_dev, c
     k.out_e = out_bf16_dev;
     k.lde = static_cast<long>(out_bf16_pitch);
     return launch_sandwich_norm(ctx, k, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" int lbk_sandwich_norm(lbk_ctx *c, float *x_dev, const float *y_dev, const float *w_post_dev, const float *w_dev, size_t rows, size_t n,
+                                 float eps, float *out_f32_dev, uint16_t *out_bf16_dev, size_t out_bf16_pitch, void *stream) {
+    return sandwich_norm(c, false, x_dev, y_dev, w_post_dev, w_dev, rows, n, eps, out_f32_dev, out_bf16_dev, out_bf16_pitch, stream);
+}
+
+extern "C" int lbk_sandwich_rms_norm(lbk_ctx *c, float *x_dev, const float *y_dev, const float *w_post_dev, const float *w_dev, size_t rows, size_t n,
+                                     float eps, float *out_f32_dev, uint16_t *out_bf16_dev, size_t out_bf16_pitch, void *stream) {
+    return sandwich_norm(c, true, x_dev, y_dev, w_post_dev, w_dev, rows, n, eps, out_f32_dev, out_bf16_dev, out_bf16_pitch, stream);
 }

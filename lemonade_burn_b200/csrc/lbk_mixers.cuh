@@ -108,7 +108,7 @@ struct RecurCall {
     const float *decay = nullptr;        // plain: [heads]
     // delta
     int taps = 1;
-    const float *conv = nullptr;         // [channels][taps], channels as in x from q_at on: q, k, v back to back
+    const float *conv = nullptr;         // [taps][channels], channels as in x from q_at on: q, k, v back to back
     void *ring = nullptr;                // [seq][taps][channels] of the compute type: the last inputs, by position modulo taps
     const float *a = nullptr;            // [rows][lda] f32, heads x dim: the projection inside softplus
     long lda = 0;
@@ -116,12 +116,20 @@ struct RecurCall {
     const float *b = nullptr;            // [rows][ldb]: logits of beta, one per head
     long ldb = 0;
     float *state = nullptr;              // [seq][heads][vdim][recur_pitch(dim)]
-    float *records = nullptr;            // recur_record_floats
+    float *records = nullptr;            // rows_of_seq >= 0: recur_record_floats
     size_t record_rows = 0;              // rows the records were sized for (more are done in several runs)
     float *o = nullptr;                  // [rows][heads * vdim]
+    // delta, one token per sequence: instead of `a` the second halves of both low-rank projections (inputs at columns
+    // a_at and g_at of x), and instead of o the gated norm per head (RMS over vdim, times norm_w, times sigmoid(gate))
+    DenseWeight a2, g2;                  // [heads * dim][rank], [heads * vdim][rank]
+    int a_at = 0, g_at = 0;
+    const float *norm_w = nullptr;
+    float eps = 0.0f;
+    void *out = nullptr;                 // [rows][heads * vdim] of the compute type, pitch ldo
+    long ldo = 0;
 };
 size_t recur_pitch(size_t dim);
-size_t recur_record_floats(bool delta, size_t rows, bool batch, size_t heads, size_t dim, size_t vdim);
+size_t recur_record_floats(bool delta, size_t rows, size_t heads, size_t dim, size_t vdim);
 constexpr size_t kRecurMaxDim = 256;
 int launch_recurrence(Ctx *ctx, const RecurCall &c, cudaStream_t st);
 

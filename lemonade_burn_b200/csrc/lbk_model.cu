@@ -99,26 +99,32 @@ int WeightLoader::shape(const std::string &name, size_t *rows, size_t *cols) con
     return LBK_OK;
 }
 
-int WeightLoader::vec(const std::string &name, size_t n, float **out, float add) {
+int WeightLoader::read(const std::string &name, size_t n, std::vector<float> &f) {
     const TensorEntry *e;
     LBK_TRY(tf.find(name, "BF16", n, 2, &e));
     std::vector<uint16_t> raw(n);
     if (pread(tf.sg.fd, raw.data(), n * 2, static_cast<off_t>(tf.sg.data0 + e->begin)) != static_cast<ssize_t>(n * 2))
         return fail(LBK_ERR_INVALID, "cannot read %s", name.c_str());
-    std::vector<float> f(n);
+    f.resize(n);
     for (size_t i = 0; i < n; ++i) {
         const uint32_t bits = static_cast<uint32_t>(raw[i]) << 16;
         memcpy(&f[i], &bits, 4);
-        f[i] += add;
     }
     tf.sg.bytes_read += n * 2;
-    tf.sg.bytes_to_device += n * 4;
+    return LBK_OK;
+}
+
+int WeightLoader::vec(const std::string &name, size_t n, float **out, float add) {
+    std::vector<float> f;
+    LBK_TRY(read(name, n, f));
+    for (float &v : f) v += add;
     return floats(f, out);
 }
 
 int WeightLoader::floats(const std::vector<float> &v, float **out) {
     LBK_TRY(dev_alloc(owner, v.size() * 4, reinterpret_cast<void **>(out)));
     LBK_CUDA(cudaMemcpy(*out, v.data(), v.size() * 4, cudaMemcpyHostToDevice));
+    tf.sg.bytes_to_device += v.size() * 4;
     return LBK_OK;
 }
 

@@ -329,6 +329,8 @@ struct WeightLoader {
 
     // rows and columns of a matrix
     int shape(const std::string &name, size_t *rows, size_t *cols) const;
+    // n values as f32 on the host
+    int read(const std::string &name, size_t n, std::vector<float> &out);
     // a vector as f32, `add` added to every value
     int vec(const std::string &name, size_t n, float **out, float add = 0.0f);
     // numbers that are not in the file
