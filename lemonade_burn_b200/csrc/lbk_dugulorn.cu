@@ -570,7 +570,8 @@ struct LayerReader {
             const DugulornLayer &src = m->layers[l.source];
             if (src.type != Mixer::Latent || !src.own || src.lat.kv_rank != s.kv_rank || src.lat.rot_dim != s.rot_dim) return bad("mixer.kv_from (a latent of the same sizes)");
         }
-        if (m->compute == LBK_COMPUTE_BF16 && s.kv_rank > 512) return fail(LBK_ERR_UNSUPPORTED, "layer %zu: latents of at most 512 values in bf16", i);
+        if (m->compute == LBK_COMPUTE_BF16 && !latent_absorb_supported(s))
+            return fail(LBK_ERR_UNSUPPORTED, "layer %zu: in bf16 latents of at most 512 values, rotated parts of at most 128", i);
         m->all_expand = m->all_expand && latent_expand_supported(s);
         std::vector<std::string> in{p + "mix.dq"};
         std::vector<size_t> rows{s.q_rank};

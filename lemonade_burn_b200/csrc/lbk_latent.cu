@@ -15,17 +15,23 @@
 //   latent_prep_kernel    a token's projections: norm of the query latent; norm of c and rotation of the key part, stored
 //                         into the cache. Angles: position * frequency in double, reduced to one turn, then sincospif.
 //   latent_rotate_kernel  rotated parts of all heads of the queries in place (expanding form)
-//   latent_absorb_kernel  W_uk,h^T q and the rotated part: a query against cache rows
-//   latent_attn_kernel    bf16: 16 or 32 heads x 64 positions at a time on mma.sync, the positions' rows staged once by
-//                         cp.async for both products; scores, softmax and sums f32, probabilities in two bf16 terms.
-//                         Slices of the positions over the blocks of the grid.
-//   latent_out_kernel     merges the slices, W_uv,h, the head's gate
+//   latent_absorb_kernel, latent_absorb_mma_kernel  W_uk,h^T q and the rotated part: a query against cache rows (32-bit, bf16)
+//   latent_attn_kernel    bf16, tcgen05: 64 positions' rows come by TMA and serve both products as they lie there. The
+//                         scores are taken transposed, positions x heads (the rows are the MMA's M side, 16 or 32 heads
+//                         its N side, so few heads cost little), and so is the output, latent dimensions x heads: the
+//                         rows again, now as the MN-major operand, times the probabilities (two bf16 terms side by side
+//                         on the N side). Both accumulate in tensor memory; the running maxima move lazily as in
+//                         lbk_attn_tc.cu. Two buffers of rows: one is filled while the other is worked on. Slices of the
+//                         positions over the blocks of the grid.
+//   latent_merge_kernel   bf16: merges the slices of up to 8 rows and multiplies by W_uv,h on mma.sync; the head's gate
+//   latent_out_kernel     32-bit: W_uv,h and the gate
 #include <algorithm>
 #include <cmath>
 
 #include "lbk_dense_dev.cuh"
 #include "lbk_mixers.cuh"
 #include "lbk_ptx.cuh"
+#include "lbk_tcgen05.cuh"
 
 namespace lbk {
 
@@ -150,16 +156,16 @@ __global__ void __launch_bounds__(256) latent_rotate_kernel(const QueryParams p)
         }
 }
 
-// One block: head blockIdx.x, 128 latent dimensions, four tokens. Threads: 16 groups of 8 dimensions x 16 shares of the
+// 32-bit. One block: head blockIdx.x, 128 latent dimensions, four tokens. Threads: 16 groups of 8 dimensions x 16 shares of the
 // head's unrotated dimensions.
 constexpr int kAbsCols = 128, kAbsTok = 4;
-template <typename T>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const QueryParams p) {
-    ptx::pdl_trigger();
-    ptx::pdl_wait();
+    using T = float;
     extern __shared__ float s_q[];                       // [kAbsTok][dim]
     __shared__ float s_part[8][kAbsTok][kAbsCols];
     const int h = blockIdx.x, c0 = blockIdx.y * kAbsCols, t0 = blockIdx.z * kAbsTok, tid = threadIdx.x;
+    ptx::pdl_trigger();
+    ptx::pdl_wait();
     const int toks = min(kAbsTok, p.rows - t0), qp = p.dp + p.rp;
     const T *q = static_cast<const T *>(p.q) + (static_cast<size_t>(t0) * p.heads + h) * qp;
     const size_t qrow = static_cast<size_t>(p.heads) * qp;
@@ -223,283 +229,556 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const QueryParams p)
     }
 }
 
+// bf16: up to 16 rows of one head x 64 latent dimensions a block, on mma.sync: rows of queries are the M side, latent
+// dimensions the N side (W_uk,h lies [dim][latent], which is the transposing load's form). Four warps, 16 dimensions each.
+constexpr int kAbRows = 16, kAbCols = 64, kAbWarps = 4;
+__global__ void __launch_bounds__(kAbWarps * 32) latent_absorb_mma_kernel(const QueryParams p) {
+    extern __shared__ __align__(16) uint8_t ab_smem[];  // queries [16][dp * 2 + 16 bytes], weights [dp][64 * 2 + 16 bytes]
+    const int h = blockIdx.x, c0 = blockIdx.y * kAbCols, t0 = blockIdx.z * kAbRows, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int toks = min(kAbRows, p.rows - t0), qp = p.dp + p.rp, qrow = p.dp * 2 + 16;
+    constexpr int kWRow = kAbCols * 2 + 16;
+    uint8_t *s_w = ab_smem + kAbRows * qrow;
+    ptx::pdl_trigger();
+    // the weights are constants: on their way while the kernel in front finishes
+    for (int i = tid; i < p.dp * 8; i += kAbWarps * 32) {
+        const int d = i >> 3, u = i & 7;
+        uint8_t *dst = s_w + d * kWRow + u * 16;
+        if (d < p.dim && c0 + u * 8 < p.uk_pitch) ptx::cp_async_16(ptx::smem_u32(dst), p.uk + (static_cast<size_t>(h) * p.dim + d) * p.uk_pitch + c0 + u * 8);
+        else *reinterpret_cast<uint4 *>(dst) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    ptx::cp_async_commit();
+    ptx::pdl_wait();
+    const uint16_t *q = static_cast<const uint16_t *>(p.q) + (static_cast<size_t>(t0) * p.heads + h) * qp;
+    const size_t next = static_cast<size_t>(p.heads) * qp;
+    for (int i = tid; i < kAbRows * (p.dp / 8); i += kAbWarps * 32) {
+        const int r = i / (p.dp / 8), u = i - r * (p.dp / 8);
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (r < toks) v = *reinterpret_cast<const uint4 *>(q + r * next + u * 8);
+        *reinterpret_cast<uint4 *>(ab_smem + r * qrow + u * 16) = v;
+    }
+    uint16_t *ql = static_cast<uint16_t *>(p.ql) + (static_cast<size_t>(t0) * p.heads + h) * p.pitch;
+    const size_t lnext = static_cast<size_t>(p.heads) * p.pitch;
+    if (blockIdx.y == 0) {
+        const int half = p.rot_dim / 2, pairs = p.rp / 2;
+        for (int e = tid; e < toks * pairs; e += kAbWarps * 32) {
+            const int r = e / pairs, i = e - r * pairs;
+            float a = 0.0f, b = 0.0f;
+            if (i < half) {
+                const float2 cs = turn(p.rot, i, p.rows_of_seq >= 0 ? p.pos[0] + t0 + r : p.pos[t0 + r]);
+                const float u = dense::bf16_f32(q[r * next + p.dp + 2 * i]), v = dense::bf16_f32(q[r * next + p.dp + 2 * i + 1]);
+                a = u * cs.x - v * cs.y;
+                b = v * cs.x + u * cs.y;
+            }
+            *reinterpret_cast<uint32_t *>(ql + r * lnext + p.kvp + 2 * i) = dense::bf16_pair(a, b);
+        }
+    }
+    ptx::cp_async_wait<0>();
+    __syncthreads();
+    const uint32_t q_lane = ptx::smem_u32(ab_smem) + ((lane & 7) + 8 * ((lane >> 3) & 1)) * qrow + (lane >> 4) * 16;
+    const uint32_t w_lane = ptx::smem_u32(s_w) + ((lane & 7) + 8 * ((lane >> 3) & 1)) * kWRow + warp * 32 + (lane >> 4) * 16;
+    float acc[2][4] = {};
+    // what lies between dim and dp in the queries is a number or another layer's, and meets zeros
+#pragma unroll 4
+    for (int k = 0; k < p.dp; k += 16) {
+        uint32_t a[4], b[4];
+        ptx::ldmatrix_x4(a, q_lane + k * 2);
+        ptx::ldmatrix_x4_trans(b, w_lane + k * kWRow);
+        ptx::mma_bf16(acc[0], a, b[0], b[1]);
+        ptx::mma_bf16(acc[1], a, b[2], b[3]);
+    }
+    const int g = lane >> 2, t = lane & 3;
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int tk = g + 8 * r, c = c0 + warp * 16 + n * 8 + 2 * t;  // columns past kv_rank have zero weights
+            if (tk < toks && c < p.kvp) *reinterpret_cast<uint32_t *>(ql + tk * lnext + c) = dense::bf16_pair(acc[n][2 * r], acc[n][2 * r + 1]);
+        }
+}
+
 // ---- attention over the latents, bf16 ---------------------------------------------------------------
-constexpr int kLKeys = 64, kLWarps = 8;
-constexpr int kLValues = 4;         // 16-dimension tiles of the latent a warp accumulates: latents of up to 512
-struct LatentLayout {
-    int krow, prow, q, ph, pl, mx, total;  // bytes
-    __host__ __device__ LatentLayout(int width, int mt) {
-        krow = width * 2 + 16;             // an odd multiple of 16: eight rows start in different bank groups
-        prow = kLKeys * 2 + 16;
-        q = 2 * kLKeys * krow;
-        ph = q + 16 * mt * krow;
-        pl = ph + 16 * mt * prow;
-        mx = pl + 16 * mt * prow;
-        total = mx + 2 * kLWarps * 16 * mt * 4;
+using namespace tc;
+
+constexpr int kLKeys = 64;          // positions at a time
+constexpr int kLPiece = kLKeys * 128;  // bytes of 64 dimensions of them (SWIZZLE_128B)
+constexpr int kLMaxPieces = 10, kLMaxLatent = 512;
+constexpr int kLGroup = 8;          // heads of four warps; warp w: TMEM lane quadrant w % 4, heads of group w / 4
+constexpr __host__ __device__ int latent_warps(int nh) { return 4 * nh / kLGroup; }  // and two more that issue copies and MMAs
+constexpr float kLRescaleStep = 8.0f;  // in units of log 2
+constexpr float kLog2e = 1.4426950408889634f;
+
+struct LatentLayout {               // bytes from a 1024-byte boundary on
+    int buf, q, p, misc, total;
+    __host__ __device__ LatentLayout(int pieces, int nh) {
+        buf = pieces * kLPiece;                // two of them
+        q = 2 * buf;                           // the heads' queries, a piece [nh rows][128 bytes]
+        p = q + pieces * nh * 128;             // probabilities, two buffers of [2 nh rows][64 positions]: high terms, then low
+        misc = p + 2 * 2 * nh * 128;           // barriers, tensor memory address, abort flag, then maxima, reference maxima, factors
+        total = misc + 256 + 3 * latent_warps(nh) * 32 * 4;
     }
 };
 struct LatentParams {
-    const uint16_t *ql, *cache;
+    CUtensorMap k;                  // bytes [sequences * cap][pitch * 2], box [64][128]
+    CUtensorMap q;                  // bytes [rows * heads][pitch * 2], box [nh][128]
     const int *pos;
-    int rows_of_seq, heads, width, kvp, pitch, cap, splits;
-    float scale;
+    int rows_of_seq, heads, width, kvp, cap, splits;
+    float scale;                    // times log2(e)
     float *part;                    // [row][head][split][kvp + 4]
     int *err_word;
 };
 
-template <int MT>  // tiles of 16 heads a block takes
-__global__ void __launch_bounds__(kLWarps * 32) latent_attn_kernel(const LatentParams p) {
+__device__ __forceinline__ void tmem_load(uint32_t at, uint32_t (&r)[8]) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+                 : "r"(at)
+                 : "memory");
+}
+__device__ __forceinline__ void tmem_store(uint32_t at, const uint32_t (&r)[8]) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"r"(at), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]),
+                 "r"(r[6]), "r"(r[7])
+                 : "memory");
+}
+// shared -> global, whole 16-byte units; the wait is until this thread's copies are complete
+__device__ __forceinline__ void bulk_store(void *dst, uint32_t src, uint32_t bytes) {
+    asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;\ncp.async.bulk.commit_group;" ::"l"(dst), "r"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void bulk_store_wait() { asm volatile("cp.async.bulk.wait_group 0;" ::: "memory"); }
+// MN-major SWIZZLE_128B operand: 64 dimensions contiguous, groups of 8 positions 1024 bytes apart, pieces of 64 dimensions
+// kLPiece apart
+__device__ __forceinline__ uint64_t smem_desc_mn(uint32_t addr) {
+    return static_cast<uint64_t>((addr & 0x3FFFFu) >> 4) | static_cast<uint64_t>(kLPiece >> 4) << 16 | static_cast<uint64_t>(1024 >> 4) << 32 | static_cast<uint64_t>(1) << 46 |
+           static_cast<uint64_t>(2) << 61;
+}
+// MMAs and commits of a whole warp: every lane comes here with the same operands and one of them, always the same, issues.
+// (Operands that are uniform over a converged warp sit in uniform registers, where the instruction wants them; under a
+// branch of one lane each would have to be moved there first, which takes longer than these small MMAs do.)
+__device__ __forceinline__ void umma(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n"
+        ".reg .pred p, e;\n"
+        "setp.ne.b32 p, %4, 0;\n"
+        "elect.sync _|e, 0xffffffff;\n"
+        "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n"
+        "}\n" ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+// Four steps of it: the operands AS and BS (16-byte units) further each time.
+template <int AS, int BS>
+__device__ __forceinline__ void umma4(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate_first) {
+    asm volatile(
+        "{\n"
+        ".reg .pred p, q, e;\n"
+        ".reg .b64 a1, a2, a3, b1, b2, b3;\n"
+        "setp.ne.b32 p, %4, 0;\n"
+        "setp.eq.b32 q, 0, 0;\n"
+        "add.u64 a1, %1, %5;\n"
+        "add.u64 a2, %1, %6;\n"
+        "add.u64 a3, %1, %7;\n"
+        "add.u64 b1, %2, %8;\n"
+        "add.u64 b2, %2, %9;\n"
+        "add.u64 b3, %2, %10;\n"
+        "elect.sync _|e, 0xffffffff;\n"
+        "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n"
+        "@e tcgen05.mma.cta_group::1.kind::f16 [%0], a1, b1, %3, q;\n"
+        "@e tcgen05.mma.cta_group::1.kind::f16 [%0], a2, b2, %3, q;\n"
+        "@e tcgen05.mma.cta_group::1.kind::f16 [%0], a3, b3, %3, q;\n"
+        "}\n" ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate_first), "n"(AS), "n"(2 * AS), "n"(3 * AS), "n"(BS), "n"(2 * BS), "n"(3 * BS)
+        : "memory");
+}
+__device__ __forceinline__ void commit(uint32_t bar) {
+    asm volatile(
+        "{\n"
+        ".reg .pred e;\n"
+        "elect.sync _|e, 0xffffffff;\n"
+        "@e tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n"
+        "}\n" ::"r"(bar)
+        : "memory");
+}
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// Over the 32 lanes, of N values each: lane l gets the maximum (or sum) of value l % N.
+template <int N, bool MAX>
+__device__ __forceinline__ float over_lanes(float (&v)[N], int lane) {
+    auto both = [](float a, float b) { return MAX ? fmaxf(a, b) : a + b; };
+#pragma unroll
+    for (int w = N / 2; w >= 1; w >>= 1) {
+        const bool up = (lane & w) != 0;
+#pragma unroll
+        for (int i = 0; i < w; ++i) v[i] = both(up ? v[i + w] : v[i], __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + w], w));
+    }
+    float t = v[0];
+#pragma unroll
+    for (int w = N; w < 32; w <<= 1) t = both(t, __shfl_xor_sync(0xffffffffu, t, w));
+    return t;
+}
+
+template <int NH>  // heads a block takes, 16 or 32
+__global__ void __launch_bounds__((latent_warps(NH) + 2) * 32, 1) latent_attn_kernel(const __grid_constant__ LatentParams p) {
+    extern __shared__ uint8_t la_raw[];
+    const uint32_t raw = ptx::smem_u32(la_raw), base = (raw + 1023u) & ~1023u;
+    uint8_t *sm = la_raw + (base - raw);
+    constexpr int HH = kLGroup, kLWarps = latent_warps(NH), kLTmaWarp = kLWarps, kLMmaWarp = kLWarps + 1;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int pieces = (p.width + 63) >> 6, blocks = (p.kvp + 127) >> 7;  // output blocks of 128 latent dimensions
+    const LatentLayout L(pieces, NH);
+    // Every barrier is a pair, by chunk parity: a wait for one chunk cannot be answered by the chunk two before it. Rows come
+    // and go in parts of two pieces (128 dimensions): scores start on the first part while the others are on their way, and
+    // a part is filled again as soon as its output block has been taken.
+    const int parts = (pieces + 1) >> 1;
+    constexpr int kParts = kLMaxPieces / 2, kFull = 0, kEmpty = 2 * kParts, kS = 4 * kParts, kP = kS + 2, kO = kS + 4;
+    auto bar = [&](int kind, int j) { return base + L.misc + (kind + (j & 1)) * 8; };
+    volatile uint32_t *s_tmem = reinterpret_cast<volatile uint32_t *>(sm + L.misc + 240);
+    volatile int *s_abort = reinterpret_cast<volatile int *>(sm + L.misc + 244);
+    float *s_max = reinterpret_cast<float *>(sm + L.misc + 256), *s_m = s_max + kLWarps * 32, *s_f = s_m + kLWarps * 32;
+    if (tid == 0) {
+        for (int i = 0; i < 2; ++i) {
+            for (int k = 0; k < kParts; ++k) {
+                ptx::mbar_init(bar(kFull + 2 * k, i), 1);
+                ptx::mbar_init(bar(kEmpty + 2 * k, i), 1);
+            }
+            ptx::mbar_init(bar(kS, i), 1);
+            ptx::mbar_init(bar(kP, i), kLWarps);
+            ptx::mbar_init(bar(kO, i), 1);
+        }
+        *s_abort = 0;
+        ptx::fence_barrier_init();
+    }
+    if (warp == kLMmaWarp) {
+        tmem_alloc(base + L.misc + 240, 512);
+        tmem_relinquish();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
     ptx::pdl_trigger();
     ptx::pdl_wait();
-    extern __shared__ __align__(16) uint8_t la_smem[];
-    const LatentLayout L(p.width, MT);
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int sp = blockIdx.x, h0 = blockIdx.y * 16 * MT, row = blockIdx.z, nh = min(16 * MT, p.heads - h0);
+    const uint32_t t_s = *s_tmem, t_o = t_s + 2 * NH;        // two buffers of scores (NH columns), then per output block 2 NH: high and low terms' sums
+    const int sp = blockIdx.x, h0 = blockIdx.y * NH, row = blockIdx.z, nh = min(NH, p.heads - h0);
     const int seq = p.rows_of_seq >= 0 ? p.rows_of_seq : row, pos = p.rows_of_seq >= 0 ? p.pos[0] + row : p.pos[row];
-    if (pos < 0 || pos >= p.cap) {
-        if (tid == 0) atomicExch(p.err_word, 7);
-        return;
-    }
-    const int total = pos + 1, per = ((total + p.splits - 1) / p.splits + kLKeys - 1) / kLKeys * kLKeys;
-    const int u0 = min(total, sp * per), u1 = min(total, u0 + per);
-    const uint16_t *kb = p.cache + static_cast<size_t>(seq) * p.cap * p.pitch;
-    const int ku = p.width / 8;                              // 16-byte units of a row
-    const uint32_t sm = ptx::smem_u32(la_smem);
-    for (int i = tid; i < 16 * MT * ku; i += kLWarps * 32) {
-        const int r = i / ku, c = i - r * ku;
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (r < nh) v = *reinterpret_cast<const uint4 *>(p.ql + (static_cast<size_t>(row) * p.heads + h0 + r) * p.pitch + c * 8);
-        *reinterpret_cast<uint4 *>(la_smem + L.q + r * L.krow + c * 16) = v;
-    }
-    auto stage = [&](int buf, int uc) {
-        const int cnt = min(kLKeys, u1 - uc);
-        for (int i = tid; i < kLKeys * ku; i += kLWarps * 32) {
-            const int r = i / ku, c = i - r * ku;
-            uint8_t *dst = la_smem + (buf * kLKeys + r) * L.krow + c * 16;
-            if (r < cnt) ptx::cp_async_16(ptx::smem_u32(dst), kb + static_cast<size_t>(uc + r) * p.pitch + c * 8);
-            else *reinterpret_cast<uint4 *>(dst) = make_uint4(0u, 0u, 0u, 0u);  // weight zero, but the bits must be numbers
-        }
-        ptx::cp_async_commit();
-    };
-    float *s_mx = reinterpret_cast<float *>(la_smem + L.mx);  // [warp][16 MT], then the same for the sums
-    const uint32_t q_lane = sm + L.q + ((lane & 7) + 8 * ((lane >> 3) & 1)) * L.krow + (lane >> 4) * 16;
-    const uint32_t k_lane0 = sm + (warp * 8 + (lane & 7)) * L.krow + (lane >> 3) * 16;
-    const uint32_t v_lane0 = sm + ((lane & 7) + 8 * ((lane >> 3) & 1)) * L.krow + (lane >> 4) * 16;
-    const uint32_t p_lane = sm + ((lane & 7) + 8 * ((lane >> 3) & 1)) * L.prow + (lane >> 4) * 16;
-    const int ksteps = p.width / 16, vtiles = p.kvp / 16;
-    float o[MT][kLValues][2][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int i = 0; i < kLValues; ++i)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) o[m][i][e][0] = o[m][i][e][1] = o[m][i][e][2] = o[m][i][e][3] = 0.0f;
-    float mrow[MT][2], lrow[MT][2];
-#pragma unroll
-    for (int m = 0; m < MT; ++m) mrow[m][0] = mrow[m][1] = -INFINITY, lrow[m][0] = lrow[m][1] = 0.0f;
-    if (u0 < u1) stage(0, u0);
-    for (int uc = u0, it = 0; uc < u1; uc += kLKeys, ++it) {
-        if (it) __syncthreads();                             // the other buffer and the probabilities have been read
-        if (uc + kLKeys < u1) {
-            stage((it & 1) ^ 1, uc + kLKeys);
-            ptx::cp_async_wait<1>();
-        } else {
-            ptx::cp_async_wait<0>();
-        }
-        __syncthreads();
-        const uint32_t boff = (it & 1) * kLKeys * L.krow;
-        float s[MT][4];
-#pragma unroll
-        for (int m = 0; m < MT; ++m) s[m][0] = s[m][1] = s[m][2] = s[m][3] = 0.0f;
-#pragma unroll 2
-        for (int kp = 0; kp < ksteps; kp += 2) {             // 32 dimensions; with an odd number of steps the last half is not used
-            uint32_t bb[4];
-            ptx::ldmatrix_x4(bb, k_lane0 + boff + kp * 32);
-#pragma unroll
-            for (int m = 0; m < MT; ++m) {
-                uint32_t a[4];
-                ptx::ldmatrix_x4(a, q_lane + m * 16 * L.krow + kp * 32);
-                ptx::mma_bf16(s[m], a, bb[0], bb[1]);
-            }
-            if (kp + 1 < ksteps) {
-#pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    uint32_t a[4];
-                    ptx::ldmatrix_x4(a, q_lane + m * 16 * L.krow + kp * 32 + 32);
-                    ptx::mma_bf16(s[m], a, bb[2], bb[3]);
-                }
-            }
-        }
-        const int key = uc + warp * 8 + 2 * t;               // this lane's keys: key, key + 1
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) s[m][e] = key + (e & 1) < u1 ? s[m][e] * p.scale : -INFINITY;
-#pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                float mx = fmaxf(s[m][2 * r], s[m][2 * r + 1]);
-                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-                if (t == 0) s_mx[warp * 16 * MT + m * 16 + g + 8 * r] = mx;
-            }
-        }
-        __syncthreads();
-        float corr[MT][2];
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                float nm = mrow[m][r];
-#pragma unroll
-                for (int w = 0; w < kLWarps; ++w) nm = fmaxf(nm, s_mx[w * 16 * MT + m * 16 + g + 8 * r]);
-                corr[m][r] = __expf(mrow[m][r] - nm);        // nm is finite: a chunk has at least one key
-                mrow[m][r] = nm;
-                const float e0 = __expf(s[m][2 * r] - nm), e1 = __expf(s[m][2 * r + 1] - nm);
-                lrow[m][r] = lrow[m][r] * corr[m][r] + e0 + e1;
-                const uint32_t hi = dense::bf16_pair(e0, e1);
-                const uint32_t lo = dense::bf16_pair(e0 - __uint_as_float(hi << 16), e1 - __uint_as_float(hi & 0xffff0000u));
-                const int at = (m * 16 + g + 8 * r) * L.prow + (warp * 8 + 2 * t) * 2;
-                *reinterpret_cast<uint32_t *>(la_smem + L.ph + at) = hi;
-                *reinterpret_cast<uint32_t *>(la_smem + L.pl + at) = lo;
-            }
-        __syncthreads();
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-            for (int i = 0; i < kLValues; ++i)
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    o[m][i][e][0] *= corr[m][0]; o[m][i][e][1] *= corr[m][0];
-                    o[m][i][e][2] *= corr[m][1]; o[m][i][e][3] *= corr[m][1];
-                }
-#pragma unroll
-        for (int ks = 0; ks < kLKeys / 16; ++ks) {
-            uint32_t ph[MT][4], pl[MT][4];
-#pragma unroll
-            for (int m = 0; m < MT; ++m) {
-                ptx::ldmatrix_x4(ph[m], p_lane + L.ph + m * 16 * L.prow + ks * 32);
-                ptx::ldmatrix_x4(pl[m], p_lane + L.pl + m * 16 * L.prow + ks * 32);
-            }
-#pragma unroll
-            for (int i = 0; i < kLValues; ++i) {
-                const int vt = warp + kLWarps * i;
-                if (vt < vtiles) {
-                    uint32_t bb[4];
-                    ptx::ldmatrix_x4_trans(bb, v_lane0 + boff + ks * 16 * L.krow + vt * 32);
-#pragma unroll
-                    for (int m = 0; m < MT; ++m) {
-                        ptx::mma_bf16(o[m][i][0], ph[m], bb[0], bb[1]);
-                        ptx::mma_bf16(o[m][i][0], pl[m], bb[0], bb[1]);
-                        ptx::mma_bf16(o[m][i][1], ph[m], bb[2], bb[3]);
-                        ptx::mma_bf16(o[m][i][1], pl[m], bb[2], bb[3]);
+    const bool pos_ok = pos >= 0 && pos < p.cap;
+    if (!pos_ok && tid == 0) atomicExch(p.err_word, 7);
+    const int total = pos_ok ? pos + 1 : 0, per = ((total + p.splits - 1) / p.splits + kLKeys - 1) / kLKeys * kLKeys;
+    const int u0 = min(total, sp * per), u1 = min(total, u0 + per), chunks = (u1 - u0 + kLKeys - 1) / kLKeys;
+    const int prow = p.kvp + 4;
+    bool ok = true;
+    if (warp == kLTmaWarp) {
+        if (lane == 0)
+            for (int j = 0; j < chunks && ok; ++j)
+                for (int k = 0; k < parts; ++k) {
+                    if (j >= 2 && !wait_bar(bar(kEmpty + 2 * k, j), ((j >> 1) - 1) & 1, s_abort)) {
+                        ok = false;
+                        break;
+                    }
+                    const int p0 = 2 * k, p1 = min(pieces, p0 + 2);
+                    ptx::mbar_arrive_expect_tx(bar(kFull + 2 * k, j), static_cast<uint32_t>((p1 - p0) * (kLPiece + (j ? 0 : NH * 128))));
+                    for (int i = p0; i < p1; ++i) {
+                        if (!j) ptx::tma_load_2d(base + L.q + i * NH * 128, &p.q, bar(kFull + 2 * k, 0), i * 128, row * p.heads + h0);
+                        ptx::tma_load_2d(base + (j & 1) * L.buf + i * kLPiece, &p.k, bar(kFull + 2 * k, j), i * 128, seq * p.cap + u0 + j * kLKeys);
                     }
                 }
+    } else if (warp == kLMmaWarp) {
+        if (chunks) {
+            // D f32, A and B bf16, M = 128. Scores: the lower 64 rows of A are the positions, the upper 64 whatever lies behind them
+            // (their lanes are not read). Output: A is MN-major (bit 15).
+            constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 4) << 24);
+            constexpr uint32_t idesc_s = idesc | (static_cast<uint32_t>(NH >> 3) << 17), idesc_o = idesc | (1u << 15) | (static_cast<uint32_t>(2 * NH >> 3) << 17);
+            const uint64_t k_desc = smem_desc_sw128(base), q_desc = smem_desc_sw128(base + L.q), v_desc = smem_desc_mn(base), p_desc = smem_desc_sw128(base + L.p);
+            const int ksteps = p.width >> 4;
+            const uint32_t u_s = __shfl_sync(0xffffffffu, t_s, 0), u_o = u_s + 2 * NH;
+            auto scores = [&](int j, int k) {                // of part k's dimensions
+                const uint64_t kd = k_desc + static_cast<uint64_t>((j & 1) * (L.buf >> 4));
+                const int end = min(ksteps, 8 * k + 8);
+                uint64_t a = kd + static_cast<uint64_t>(2 * k * (kLPiece >> 4)), b = q_desc + static_cast<uint64_t>(2 * k * (NH * 128 >> 4));
+                int st = 8 * k;
+#pragma unroll
+                for (int i = 0; i < 2; ++i)                  // pieces of 64 dimensions
+                    if (st + 4 <= end) {
+                        umma4<2, 2>(u_s + (j & 1) * NH, a, b, idesc_s, (k | i) ? 1u : 0u);
+                        a += kLPiece >> 4;
+                        b += NH * 128 >> 4;
+                        st += 4;
+                    }
+                for (; st < end; ++st)
+                    umma(u_s + (j & 1) * NH, kd + static_cast<uint64_t>((st >> 2) * (kLPiece >> 4) + (st & 3) * 2),
+                         q_desc + static_cast<uint64_t>((st >> 2) * (NH * 128 >> 4) + (st & 3) * 2), idesc_s, st ? 1u : 0u);
+                if (k == parts - 1) commit(bar(kS, j));
+            };
+            auto values = [&](int j) {
+                const uint64_t vd = v_desc + static_cast<uint64_t>((j & 1) * (L.buf >> 4)), pd = p_desc + static_cast<uint64_t>((j & 1) * (2 * NH * 128 >> 4));
+                for (int k = 0; k < parts; ++k) {
+                    if (k < blocks) umma4<(2048 >> 4), 2>(u_o + k * 2 * NH, vd + static_cast<uint64_t>(k * (2 * kLPiece >> 4)), pd, idesc_o, j ? 1u : 0u);  // 16 positions a step
+                    commit(bar(kEmpty + 2 * k, j));
+                }
+                commit(bar(kO, j));
+            };
+            // Values of chunk nv as soon as its probabilities are there, else scores of chunk ns's next part as soon as that
+            // is, never more than two chunks apart. So scores of j + 1 go after values of j - 1: the probabilities of j - 1
+            // mean that its scores have been read (the buffer is j + 1's), and scores of j + 1 mean that the probabilities
+            // of j - 1 have been (the same for theirs).
+            int ns = 0, nk = 0, nv = 0;
+            uint32_t idle = 0;
+            while (nv < chunks) {
+                if (nv < ns && __all_sync(0xffffffffu, ptx::mbar_test_wait(bar(kP, nv), (nv >> 1) & 1))) {
+                    tc_fence_after();
+                    values(nv++);
+                    idle = 0;
+                } else if (ns < chunks && ns <= nv + 1 && __all_sync(0xffffffffu, ptx::mbar_test_wait(bar(kFull + 2 * nk, ns), (ns >> 1) & 1))) {
+                    scores(ns, nk);
+                    if (++nk == parts) {
+                        nk = 0;
+                        ++ns;
+                    }
+                    idle = 0;
+                } else if (__any_sync(0xffffffffu, *s_abort || ++idle > kTcWaitLimit)) {
+                    *s_abort = 1;
+                    ok = false;
+                    break;
+                }
             }
         }
+    } else {
+        auto wait_all = [&](uint32_t b, uint32_t parity) { return __all_sync(0xffffffffu, wait_bar(b, parity, s_abort)) != 0; };
+        const int quad = warp & 3, group = warp >> 2;        // positions are in quadrants 0 and 1; all four hold latent dimensions
+        const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
+        auto meet = [&]() { asm volatile("bar.sync %0, 128;" ::"r"(1 + group) : "memory"); };  // the four warps of a group
+        float *w_m = s_m + warp * 32, *w_f = s_f + warp * 32, *g_max = s_max + group * 4 * 32;
+        float m = -1e30f, l = 0.0f;                          // of head lane % HH: the maximum probabilities are scaled with, this warp's share of the sum
+        // Every warp comes to the meeting of a chunk and to the one after the loop whatever a wait returned: a warp whose
+        // wait gave up skips the work, never the meetings.
+        for (int j = 0; j < chunks; ++j) {
+            const int key = u0 + j * kLKeys + quad * 32 + lane;
+            float s[HH], v[HH];
+            if (quad < 2) {
+                if (ok && !wait_all(bar(kS, j), (j >> 1) & 1)) ok = false;
+                if (ok) {
+                    tc_fence_after();
+                    uint32_t r[HH];
+                    tmem_load(t_s + (j & 1) * NH + group * HH + lanes, r);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int i = 0; i < HH; ++i) s[i] = v[i] = key < u1 ? __uint_as_float(r[i]) * p.scale : -INFINITY;
+                    g_max[((j & 1) * 2 + quad) * 32 + lane] = over_lanes<HH, true>(v, lane);
+                }
+            }
+            meet();  // the maxima's place of this parity is written again two chunks later, after the next meeting
+            if (!ok) continue;
+            const float mx = fmaxf(g_max[(j & 1) * 2 * 32 + lane], g_max[((j & 1) * 2 + 1) * 32 + lane]);  // finite: a chunk has a position
+            const float nm = mx > m + kLRescaleStep ? mx : m, corr = ex2(m - nm);
+            const bool moved = __any_sync(0xffffffffu, nm != m) && j > 0;  // the same in the four warps
+            m = nm;
+            w_m[lane] = nm;
+            w_f[lane] = corr;
+            __syncwarp();
+            if (moved) {                                     // nothing adds to the output before all warps say that their probabilities are ready
+                if (!wait_all(bar(kO, j - 1), ((j - 1) >> 1) & 1)) {
+                    ok = false;
+                    continue;
+                }
+                tc_fence_after();
+                for (int c = 0; c < 2 * blocks; ++c) {       // high and low terms of every block
+                    uint32_t r[HH];
+                    tmem_load(t_o + c * NH + group * HH + lanes, r);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int i = 0; i < HH; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * w_f[i]);
+                    tmem_store(t_o + c * NH + group * HH + lanes, r);
+                }
+                tmem_st_wait();
+            }
+            if (quad < 2) {
+                // position k of head i: row i, 16-byte unit k / 8 XOR-ed with i % 8
+                const int k = quad * 32 + lane;
+                uint8_t *pp = sm + L.p + (j & 1) * 2 * NH * 128 + group * HH * 128 + (k & 7) * 2;
+#pragma unroll
+                for (int i = 0; i < HH; ++i) {
+                    const float e = ex2(s[i] - w_m[i]);
+                    v[i] = e;
+                    const uint32_t hi = dense::bf16_pair(e, 0.0f);
+                    uint8_t *at = pp + i * 128 + (((k >> 3) ^ (i & 7)) << 4);
+                    *reinterpret_cast<uint16_t *>(at) = static_cast<uint16_t>(hi);
+                    *reinterpret_cast<uint16_t *>(at + NH * 128) = dense::f32_bf16(e - __uint_as_float(hi << 16));
+                }
+                l = l * corr + over_lanes<HH, false>(v, lane);
+                if (key >= total && group == 0) {             // nothing has been written there: its weight is zero, but the bits must be numbers
+                    for (int i = 0; i < pieces; ++i)
+#pragma unroll
+                        for (int u = 0; u < 8; ++u) *reinterpret_cast<uint4 *>(sm + (j & 1) * L.buf + i * kLPiece + k * 128 + u * 16) = make_uint4(0u, 0u, 0u, 0u);
+                }
+                ptx::fence_proxy_async();
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) ptx::mbar_arrive(bar(kP, j));
+        }
+        if (ok && chunks && !wait_all(bar(kO, chunks - 1), ((chunks - 1) >> 1) & 1)) ok = false;
+        tc_fence_after();
+        // this slice's sums and, unscaled, the weighted latents (an empty slice: no weight, zeros)
+        w_f[lane] = l;
+        float *out = reinterpret_cast<float *>(sm) + group * HH * p.kvp;  // every copy and MMA has finished: the rows' buffers are free
+        for (int db = 0; db < blocks; ++db) {
+            uint32_t r[HH], lo[HH];
+#pragma unroll
+            for (int i = 0; i < HH; ++i) r[i] = lo[i] = 0;
+            if (ok && chunks) {
+                tmem_load(t_o + db * 2 * NH + group * HH + lanes, r);
+                tmem_load(t_o + db * 2 * NH + NH + group * HH + lanes, lo);
+                tmem_ld_wait();
+            }
+            const int d = db * 128 + quad * 32 + lane;
+            if (d < p.kvp)
+#pragma unroll
+                for (int i = 0; i < HH; ++i) out[i * p.kvp + d] = __uint_as_float(r[i]) + __uint_as_float(lo[i]);
+        }
+        ptx::fence_proxy_async();
+        meet();
+        if (quad == 0 && lane < HH && group * HH + lane < nh) {
+            float *dst = p.part + ((static_cast<size_t>(row) * p.heads + h0 + group * HH + lane) * p.splits + sp) * prow;
+            bulk_store(dst, ptx::smem_u32(out + lane * p.kvp), static_cast<uint32_t>(p.kvp) * 4);
+            dst[p.kvp] = chunks ? m / kLog2e : -INFINITY;
+            dst[p.kvp + 1] = w_f[lane] + w_f[32 + lane];  // this warp's and the next one's
+            bulk_store_wait();
+        }
+        tc_fence_before();
     }
-    // this slice's sums and, unscaled, the weighted latents
-    float *s_l = s_mx + kLWarps * 16 * MT;
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            float v = lrow[m][r];
-            v += __shfl_xor_sync(0xffffffffu, v, 1);
-            v += __shfl_xor_sync(0xffffffffu, v, 2);
-            if (t == 0) s_l[warp * 16 * MT + m * 16 + g + 8 * r] = v;
-        }
+    if (!ok && lane == 0) atomicExch(p.err_word, 5);
     __syncthreads();
-    const int prow = p.kvp + 4;
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            const int hr = m * 16 + g + 8 * r;
-            if (hr >= nh) continue;
-            float *dst = p.part + ((static_cast<size_t>(row) * p.heads + h0 + hr) * p.splits + sp) * prow;
-#pragma unroll
-            for (int i = 0; i < kLValues; ++i) {
-                const int vt = warp + kLWarps * i;
-                if (vt < vtiles)
-#pragma unroll
-                    for (int e = 0; e < 2; ++e) *reinterpret_cast<float2 *>(dst + vt * 16 + e * 8 + 2 * t) = make_float2(o[m][i][e][2 * r], o[m][i][e][2 * r + 1]);
-            }
-            if (warp == 0 && t == 0) {
-                float sum = 0.0f;
-#pragma unroll
-                for (int w = 0; w < kLWarps; ++w) sum += s_l[w * 16 * MT + hr];
-                dst[p.kvp] = mrow[m][r];                     // -inf for an empty slice: the merge gives it no weight
-                dst[p.kvp + 1] = sum;
-            }
-        }
+    if (warp == kLMmaWarp) {
+        tc_fence_after();
+        tmem_dealloc(t_s, 512);
+    }
 }
 
 // ---- out: merge, W_uv, gate -----------------------------------------------------------------------------
 struct OutParams {
-    const float *part;              // slices, or (splits = 0) the weighted latents themselves, [row][heads][kv_rank]
+    const float *part;              // slices, or (32-bit) the weighted latents themselves, [row][heads][kv_rank]
     int rows, heads, splits, vdim, kv_rank, kvp;
     const uint16_t *uv;
-    int uv_pitch;
+    int uv_pitch, vrows;            // vrows: value dimensions a block takes (a multiple of 16)
     const float *gate;
     long ldg, ldo;
     void *out;
 };
+constexpr int kMergeTok = 8;        // the MMA's N side
+__global__ void __launch_bounds__(256) latent_merge_kernel(const OutParams p) {
+    __shared__ __align__(16) float s_sum[8][kLMaxLatent];    // [warp][latent]
+    __shared__ __align__(16) uint16_t s_x[kMergeTok][kLMaxLatent + 32];  // eight rows start in different bank groups
+    ptx::pdl_trigger();
+    const int h = blockIdx.x, e0 = blockIdx.y * p.vrows, t0 = blockIdx.z * kMergeTok, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int toks = min(kMergeTok, p.rows - t0), prow = p.kvp + 4;
+    // the weights are constants: the warp's first 16 rows are on their way while the kernel in front finishes
+    const int g = lane >> 2, t = lane & 3, e_end = min(p.vdim, e0 + p.vrows);
+    constexpr int kAhead = 8;
+    uint4 wl[kAhead], wh[kAhead];
+    auto weights = [&](int r0, int c0) {                     // 32 columns each: 16 bytes a lane are two MMAs' operands
+        const uint16_t *lo = p.uv + static_cast<size_t>(h * p.vdim + min(r0 + g, p.vdim - 1)) * p.uv_pitch + t * 8;
+        const uint16_t *hi = p.uv + static_cast<size_t>(h * p.vdim + min(r0 + g + 8, p.vdim - 1)) * p.uv_pitch + t * 8;
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i)
+            if (c0 + 32 * i < p.uv_pitch) {
+                wl[i] = *reinterpret_cast<const uint4 *>(lo + c0 + 32 * i);
+                wh[i] = *reinterpret_cast<const uint4 *>(hi + c0 + 32 * i);
+            }
+    };
+    if (e0 + warp * 16 < e_end) weights(e0 + warp * 16, 0);
+    ptx::pdl_wait();
+    // a warp or several for each row, every so many slices; what lies between kv_rank and kvp is zero
+    int share = 8;
+    while (share * toks > 8) share >>= 1;
+    const int tok = warp / share, sub = warp - tok * share;
+    if (tok < toks) {
+        const float *part = p.part + (static_cast<size_t>(t0 + tok) * p.heads + h) * p.splits * prow;
+        const int sa = lane, sb = lane + 32;                 // at most 64 slices
+        const float ma = sa < p.splits ? part[static_cast<size_t>(sa) * prow + p.kvp] : -INFINITY, mb = sb < p.splits ? part[static_cast<size_t>(sb) * prow + p.kvp] : -INFINITY;
+        const float la = sa < p.splits ? part[static_cast<size_t>(sa) * prow + p.kvp + 1] : 0.0f, lb = sb < p.splits ? part[static_cast<size_t>(sb) * prow + p.kvp + 1] : 0.0f;
+        float4 a[kLMaxLatent / 128];
+#pragma unroll
+        for (int j = 0; j < kLMaxLatent / 128; ++j) a[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        float wa = 0.0f, wb = 0.0f;
+        constexpr int kBatch = 5;                            // slices whose values are in flight together
+        for (int s0 = sub; s0 < p.splits; s0 += kBatch * share) {
+            float4 v[kBatch][kLMaxLatent / 128];
+#pragma unroll
+            for (int k = 0; k < kBatch; ++k)
+#pragma unroll
+                for (int j = 0; j < kLMaxLatent / 128; ++j) {
+                    const int s = s0 + k * share;
+                    v[k][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (s < p.splits && lane * 4 + 128 * j < p.kvp) v[k][j] = *reinterpret_cast<const float4 *>(part + static_cast<size_t>(s) * prow + lane * 4 + 128 * j);
+                }
+            if (s0 == sub) {
+                float mx = fmaxf(ma, mb);
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+                wa = ma == -INFINITY ? 0.0f : __expf(ma - mx);
+                wb = mb == -INFINITY ? 0.0f : __expf(mb - mx);
+                float sum = wa * la + wb * lb;
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+                wa /= sum;
+                wb /= sum;
+            }
+#pragma unroll
+            for (int k = 0; k < kBatch; ++k) {
+                const int s = s0 + k * share;
+                const float x = __shfl_sync(0xffffffffu, s < 32 ? wa : wb, s & 31), w = s < p.splits ? x : 0.0f;
+#pragma unroll
+                for (int j = 0; j < kLMaxLatent / 128; ++j) {
+                    a[j].x = fmaf(w, v[k][j].x, a[j].x); a[j].y = fmaf(w, v[k][j].y, a[j].y); a[j].z = fmaf(w, v[k][j].z, a[j].z); a[j].w = fmaf(w, v[k][j].w, a[j].w);
+                }
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < kLMaxLatent / 128; ++j) {
+            if (share == 1) dense::put4(&s_x[tok][lane * 4 + 128 * j], a[j]);
+            else *reinterpret_cast<float4 *>(&s_sum[warp][lane * 4 + 128 * j]) = a[j];
+        }
+    }
+    if (share > 1) __syncthreads();
+    for (int i = tid; i < kMergeTok * p.uv_pitch; i += 256) {
+        const int tk = i / p.uv_pitch, c = i - tk * p.uv_pitch;
+        if (tk < toks && share == 1) continue;               // already there
+        float v = 0.0f;
+        if (tk < toks)
+            for (int k = 0; k < share; ++k) v += s_sum[tk * share + k][c];
+        s_x[tk][c] = dense::f32_bf16(v);
+    }
+    __syncthreads();
+    for (int r0 = e0 + warp * 16; r0 < e_end; r0 += 128) {
+        float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        for (int c0 = 0; c0 < p.uv_pitch; c0 += 32 * kAhead) {
+            if (c0 || r0 != e0 + warp * 16) weights(r0, c0);
+#pragma unroll
+            for (int i = 0; i < kAhead; ++i)
+                if (c0 + 32 * i < p.uv_pitch) {
+                    const uint4 b = *reinterpret_cast<const uint4 *>(&s_x[g][c0 + 32 * i + t * 8]);
+                    const uint32_t a0[4] = {wl[i].x, wh[i].x, wl[i].y, wh[i].y}, a1[4] = {wl[i].z, wh[i].z, wl[i].w, wh[i].w};
+                    ptx::mma_bf16(acc, a0, b.x, b.y);        // both operands with the same order of columns
+                    ptx::mma_bf16(acc, a1, b.z, b.w);
+                }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int tk = 2 * t + (i & 1), e = r0 + g + 8 * (i >> 1);
+            if (tk < toks && e < e_end)
+                static_cast<uint16_t *>(p.out)[static_cast<size_t>(t0 + tk) * p.ldo + static_cast<size_t>(h) * p.vdim + e] =
+                    dense::f32_bf16(acc[i] * dense::sigmoid(p.gate[static_cast<size_t>(t0 + tk) * p.ldg + h]));
+        }
+    }
+}
+
 constexpr int kOutTok = 4, kOutRows = 32;
-template <typename T>
 __global__ void __launch_bounds__(256) latent_out_kernel(const OutParams p) {
     ptx::pdl_trigger();
     ptx::pdl_wait();
-    extern __shared__ float s_dyn[];                         // [kOutTok][uv_pitch], [splits] weights
-    __shared__ float4 s_half[128];                           // the second half of the slices' sum (latents of up to 512)
-    float *s_w = s_dyn + kOutTok * p.uv_pitch;
+    extern __shared__ float s_dyn[];                         // [kOutTok][uv_pitch]
     const int h = blockIdx.x, e0 = blockIdx.y * kOutRows, t0 = blockIdx.z * kOutTok, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int toks = min(kOutTok, p.rows - t0);
-    for (int t = 0; t < kOutTok; ++t) {
-        float *x = s_dyn + t * p.uv_pitch;
-        if (t >= toks) {
-            for (int i = tid; i < p.uv_pitch; i += 256) x[i] = 0.0f;
-            continue;
-        }
-        const size_t rh = static_cast<size_t>(t0 + t) * p.heads + h;
-        if (p.splits == 0) {
-            for (int i = tid; i < p.uv_pitch; i += 256) x[i] = i < p.kv_rank ? p.part[rh * p.kv_rank + i] : 0.0f;
-            continue;
-        }
-        const int prow = p.kvp + 4;
-        const float *part = p.part + rh * p.splits * prow;
-        // every warp works the weights out for itself
-        float mx = -INFINITY, sum = 0.0f;
-        for (int s = lane; s < p.splits; s += 32) mx = fmaxf(mx, part[static_cast<size_t>(s) * prow + p.kvp]);
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-        __syncthreads();                                     // the weights of the token before have been read
-        for (int s = lane; s < p.splits; s += 32) {
-            const float m = part[static_cast<size_t>(s) * prow + p.kvp];
-            const float w = m == -INFINITY ? 0.0f : __expf(m - mx);
-            if (warp == 0) s_w[s] = w;
-            sum += w * part[static_cast<size_t>(s) * prow + p.kvp + 1];
-        }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        __syncthreads();
-        const float inv = 1.0f / sum;
-        // four values a thread, every second slice; what lies between kv_rank and kvp is zero
-        const int i = (tid & 127) * 4, half = tid >> 7;
-        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (i < p.kvp) {
-#pragma unroll 16
-            for (int s = half; s < p.splits; s += 2) {
-                const float4 v = *reinterpret_cast<const float4 *>(part + static_cast<size_t>(s) * prow + i);
-                const float w = s_w[s];
-                a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
-            }
-        }
-        if (half) s_half[tid & 127] = a;
-        __syncthreads();
-        if (!half && i < p.uv_pitch) {
-            const float4 b = s_half[tid];
-            *reinterpret_cast<float4 *>(x + i) = make_float4((a.x + b.x) * inv, (a.y + b.y) * inv, (a.z + b.z) * inv, (a.w + b.w) * inv);
-        }
+    for (int i = tid; i < kOutTok * p.uv_pitch; i += 256) {
+        const int t = i / p.uv_pitch, c = i - t * p.uv_pitch;
+        s_dyn[i] = t < toks && c < p.kv_rank ? p.part[(static_cast<size_t>(t0 + t) * p.heads + h) * p.kv_rank + c] : 0.0f;
     }
     __syncthreads();
     for (int r = warp; r < kOutRows; r += 8) {
@@ -507,42 +786,39 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const OutParams p) {
         if (e >= p.vdim) break;
         const uint16_t *w = p.uv + static_cast<size_t>(h * p.vdim + e) * p.uv_pitch;
         float acc[kOutTok] = {};
-        for (int i = lane * 8; i < p.uv_pitch; i += 256) {
-            const uint4 v = *reinterpret_cast<const uint4 *>(w + i);
-            const uint32_t wv[4] = {v.x, v.y, v.z, v.w};
+        for (int i = lane; i < p.uv_pitch; i += 32) {
+            const float wv = dense::bf16_f32(w[i]);
 #pragma unroll
-            for (int t = 0; t < kOutTok; ++t) {
-                const float4 a = *reinterpret_cast<const float4 *>(s_dyn + t * p.uv_pitch + i), b = *reinterpret_cast<const float4 *>(s_dyn + t * p.uv_pitch + i + 4);
-                const float x[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
-#pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    acc[t] = fmaf(__uint_as_float(wv[k] << 16), x[2 * k], acc[t]);
-                    acc[t] = fmaf(__uint_as_float(wv[k] & 0xffff0000u), x[2 * k + 1], acc[t]);
-                }
-            }
+            for (int t = 0; t < kOutTok; ++t) acc[t] = fmaf(wv, s_dyn[t * p.uv_pitch + i], acc[t]);
         }
 #pragma unroll
         for (int t = 0; t < kOutTok; ++t) {
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], o);
             if (lane == 0 && t < toks)
-                dense::put(static_cast<T *>(p.out) + static_cast<size_t>(t0 + t) * p.ldo + static_cast<size_t>(h) * p.vdim + e,
-                           acc[t] * dense::sigmoid(p.gate[static_cast<size_t>(t0 + t) * p.ldg + h]));
+                static_cast<float *>(p.out)[static_cast<size_t>(t0 + t) * p.ldo + static_cast<size_t>(h) * p.vdim + e] =
+                    acc[t] * dense::sigmoid(p.gate[static_cast<size_t>(t0 + t) * p.ldg + h]);
         }
     }
 }
 
 constexpr size_t kMaxSplits = 64;
 constexpr int kLatentSmem = 227 * 1024;
+static_assert(kMaxSplits <= 64, "a lane of the merge holds two slices' weights");
 
-bool latent_mma_supported(const LatentShape &s) {
-    return s.kvp() <= kLWarps * kLValues * 16 && LatentLayout(static_cast<int>(s.kvp() + s.rp()), 1).total <= kLatentSmem;
+// The scores' operand is read 128 rows at a time (half of them belong to what lies behind a piece), the output's in blocks of
+// two pieces: all of it has to be the block's own shared memory.
+int latent_smem(const LatentShape &s, int nh) {
+    const int pieces = static_cast<int>((s.kvp() + s.rp() + 63) / 64), own = LatentLayout(pieces, nh).total;
+    const int scores = (2 * pieces + 1) * kLPiece, values = pieces * kLPiece + static_cast<int>((s.kvp() + 127) / 128) * 2 * kLPiece;
+    return std::max(own, std::max(scores, values)) + 1024;
 }
 
 int latent_init(Ctx *ctx) {
     const int most = static_cast<int>(ctx->smem_optin) < kLatentSmem ? static_cast<int>(ctx->smem_optin) : kLatentSmem;
-    LBK_CUDA(cudaFuncSetAttribute(latent_attn_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
-    LBK_CUDA(cudaFuncSetAttribute(latent_attn_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
+    LBK_CUDA(cudaFuncSetAttribute(latent_absorb_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
+    LBK_CUDA(cudaFuncSetAttribute(latent_attn_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
+    LBK_CUDA(cudaFuncSetAttribute(latent_attn_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
     return LBK_OK;
 }
 const InitHook kInitLatent(latent_init);
@@ -637,8 +913,13 @@ int launch_latent_absorbed(Ctx *ctx, const LatentAttnCall &c, cudaStream_t st) {
     if (c.rows > 65535) return fail(LBK_ERR_UNSUPPORTED, "at most 65535 rows per call");
     const bool f32 = c.compute == LBK_COMPUTE_F32;
     const QueryParams qp = query_params(c);
-    const dim3 agrid(static_cast<unsigned>(c.s.heads), static_cast<unsigned>((c.s.kvp() + kAbsCols - 1) / kAbsCols), static_cast<unsigned>((c.rows + kAbsTok - 1) / kAbsTok));
-    LBK_CUDA(launch_chained(f32 ? latent_absorb_kernel<float> : latent_absorb_kernel<uint16_t>, agrid, dim3(256), kAbsTok * c.s.dim * sizeof(float), st, qp));
+    if (f32) {
+        const dim3 grid(static_cast<unsigned>(c.s.heads), static_cast<unsigned>((c.s.kvp() + kAbsCols - 1) / kAbsCols), static_cast<unsigned>((c.rows + kAbsTok - 1) / kAbsTok));
+        LBK_CUDA(launch_chained(latent_absorb_kernel, grid, dim3(256), kAbsTok * c.s.dim * sizeof(float), st, qp));
+    } else {
+        const dim3 grid(static_cast<unsigned>(c.s.heads), static_cast<unsigned>((c.s.kvp() + kAbCols - 1) / kAbCols), static_cast<unsigned>((c.rows + kAbRows - 1) / kAbRows));
+        LBK_CUDA(launch_chained(latent_absorb_mma_kernel, grid, dim3(kAbWarps * 32), kAbRows * (c.s.dp() * 2 + 16) + c.s.dp() * (kAbCols * 2 + 16), st, qp));
+    }
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;
     OutParams op{};
@@ -675,38 +956,51 @@ int launch_latent_absorbed(Ctx *ctx, const LatentAttnCall &c, cudaStream_t st) {
         a.ldo = static_cast<long>(c.s.heads * c.s.kv_rank);
         LBK_TRY(launch_attn_window(ctx, a, st));
     } else {
-        if (!latent_mma_supported(c.s)) return fail(LBK_ERR_UNSUPPORTED, "latent attention in bf16: latents of at most 512 values");
+        const int nh = c.s.heads > 16 ? 32 : 16;
+        if (!latent_absorb_supported(c.s)) return fail(LBK_ERR_UNSUPPORTED, "latent attention in bf16: latents of at most %d values, rotated parts of at most 128", kLMaxLatent);
         LatentParams p{};
-        p.ql = static_cast<const uint16_t *>(c.ql);
-        p.cache = static_cast<const uint16_t *>(c.cache);
+        const size_t pitch = c.s.pitch() * 2, seqs = c.rows_of_seq >= 0 ? static_cast<size_t>(c.rows_of_seq) + 1 : c.rows;
+        LBK_TRY(encode_bytes_map(&p.k, c.cache, pitch, seqs * c.cap, pitch, 128, kLKeys));
+        LBK_TRY(encode_bytes_map(&p.q, c.ql, pitch, c.rows * c.s.heads, pitch, 128, nh));
         p.pos = c.pos;
         p.rows_of_seq = c.rows_of_seq;
         p.heads = qp.heads;
         p.width = static_cast<int>(c.s.kvp() + c.s.rp());
         p.kvp = qp.kvp;
-        p.pitch = qp.pitch;
         p.cap = static_cast<int>(c.cap);
-        p.scale = c.scale;
+        p.scale = c.scale * kLog2e;
         p.part = c.scratch;
         p.err_word = ctx->err_word;
-        const bool two = c.s.heads > 16 && LatentLayout(p.width, 2).total <= kLatentSmem;
-        const size_t tiles = (c.s.heads + (two ? 31 : 15)) / (two ? 32 : 16);
+        const size_t tiles = (c.s.heads + nh - 1) / nh;
         // about one block per SM: as many slices as that leaves
         const size_t want = static_cast<size_t>(ctx->sm_count) / (c.rows * tiles);
         p.splits = static_cast<int>(want < 1 ? 1 : want < c.splits ? want : c.splits);
         op.splits = p.splits;
         const dim3 grid(static_cast<unsigned>(p.splits), static_cast<unsigned>(tiles), static_cast<unsigned>(c.rows));
-        LBK_CUDA(launch_chained(two ? latent_attn_kernel<2> : latent_attn_kernel<1>, grid, dim3(kLWarps * 32), static_cast<size_t>(LatentLayout(p.width, two ? 2 : 1).total), st, p));
+        LBK_CUDA(launch_chained(nh == 32 ? latent_attn_kernel<32> : latent_attn_kernel<16>, grid, dim3(static_cast<unsigned>(latent_warps(nh) + 2) * 32), static_cast<size_t>(latent_smem(c.s, nh)), st, p));
         LBK_CUDA(cudaGetLastError());
         ctx->launches++;
+        // a block for eight rows of a head, or for fewer value dimensions of them when that leaves SMs idle
+        const size_t ttiles = (c.rows + kMergeTok - 1) / kMergeTok, vtiles = (c.s.vdim + 15) / 16;
+        size_t parts = static_cast<size_t>(ctx->sm_count) / (c.s.heads * ttiles);
+        parts = parts < 1 ? 1 : parts > vtiles ? vtiles : parts;
+        op.vrows = static_cast<int>((vtiles + parts - 1) / parts * 16);
+        const dim3 mgrid(static_cast<unsigned>(c.s.heads), static_cast<unsigned>((c.s.vdim + op.vrows - 1) / op.vrows), static_cast<unsigned>(ttiles));
+        LBK_CUDA(launch_chained(latent_merge_kernel, mgrid, dim3(256), 0, st, op));
+        LBK_CUDA(cudaGetLastError());
+        ctx->launches++;
+        return LBK_OK;
     }
     const dim3 ogrid(static_cast<unsigned>(c.s.heads), static_cast<unsigned>((c.s.vdim + kOutRows - 1) / kOutRows), static_cast<unsigned>((c.rows + kOutTok - 1) / kOutTok));
-    LBK_CUDA(launch_chained(f32 ? latent_out_kernel<float> : latent_out_kernel<uint16_t>, ogrid, dim3(256), (kOutTok * c.uv.pitch + kMaxSplits) * sizeof(float), st, op));
+    LBK_CUDA(launch_chained(latent_out_kernel, ogrid, dim3(256), kOutTok * c.uv.pitch * sizeof(float), st, op));
     LBK_CUDA(cudaGetLastError());
     ctx->launches++;
     return LBK_OK;
 }
 
+bool latent_absorb_supported(const LatentShape &s) {
+    return s.kvp() <= kLMaxLatent && (s.kvp() + s.rp() + 63) / 64 <= kLMaxPieces && latent_smem(s, 32) <= kLatentSmem;
+}
 bool latent_expand_supported(const LatentShape &s) { return (s.dp() + 63) / 64 + (s.rp() + 63) / 64 <= 3 && s.vp() <= 128; }
 
 int launch_latent_expanded(Ctx *ctx, const LatentAttnCall &c, cudaStream_t st) {

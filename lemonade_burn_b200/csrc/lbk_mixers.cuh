@@ -85,6 +85,7 @@ struct LatentAttnCall {
 };
 size_t latent_splits(size_t cap);
 size_t latent_scratch(const Ctx *ctx, size_t rows, const LatentShape &s, size_t splits);
+bool latent_absorb_supported(const LatentShape &s);  // bf16; 32-bit has no such limit
 bool latent_expand_supported(const LatentShape &s);
 int launch_latent_absorbed(Ctx *ctx, const LatentAttnCall &c, cudaStream_t st);
 int launch_latent_expanded(Ctx *ctx, const LatentAttnCall &c, cudaStream_t st);
