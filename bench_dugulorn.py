@@ -92,6 +92,9 @@ def kernels(torch, ctx, peaks):
                     calls = [(lambda w=w: chk(lib.lbk_dense_linear_act(h, 0, x.data_ptr(), c, m, w.data_ptr(), c, r, c, bias.data_ptr() if kind == 1 else None, act, to,
                                                                        out.data_ptr(), r, int(f32), st()))) for w in ws]
                 us = graph_us(torch, calls * (1 if m < 2048 else 5))
+                if not gated:  # the like kernel at equal size: the same projection with Pefolix's epilogue
+                    plain = [(lambda w=w: chk(lib.lbk_dense_linear(h, 0, x.data_ptr(), c, m, w.data_ptr(), c, wr, c, 0, r, 0, out.data_ptr(), r, int(f32), None, 0, st()))) for w in ws]
+                    add("projection", f"{c} -> {r}, {m} tokens", "Pefolix", graph_us(torch, plain * (1 if m < 2048 else 5)), nbytes + m * c * 2 + out.numel() * out.element_size(), 2.0 * m * wr * c)
                 add("projection", f"{name} {c} -> {r}, {m} tokens", "Pefolix" if gated else "Dugulorn", us, nbytes + m * c * 2 + out.numel() * out.element_size(), 2.0 * m * wr * c)
                 del ws
         torch.cuda.empty_cache()

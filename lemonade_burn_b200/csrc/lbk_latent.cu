@@ -338,11 +338,12 @@ __device__ __forceinline__ void tmem_store(uint32_t at, const uint32_t (&r)[8]) 
                  "r"(r[6]), "r"(r[7])
                  : "memory");
 }
-// shared -> global, whole 16-byte units; the wait is until this thread's copies are complete
+// shared -> global, whole 16-byte units; the wait is until this thread's copies have been read from shared memory (they are
+// complete when the grid is)
 __device__ __forceinline__ void bulk_store(void *dst, uint32_t src, uint32_t bytes) {
     asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;\ncp.async.bulk.commit_group;" ::"l"(dst), "r"(src), "r"(bytes) : "memory");
 }
-__device__ __forceinline__ void bulk_store_wait() { asm volatile("cp.async.bulk.wait_group 0;" ::: "memory"); }
+__device__ __forceinline__ void bulk_store_wait() { asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory"); }
 // MN-major SWIZZLE_128B operand: 64 dimensions contiguous, groups of 8 positions 1024 bytes apart, pieces of 64 dimensions
 // kLPiece apart
 __device__ __forceinline__ uint64_t smem_desc_mn(uint32_t addr) {
@@ -591,15 +592,25 @@ __global__ void __launch_bounds__((latent_warps(NH) + 2) * 32, 1) latent_attn_ke
             if (quad < 2) {
                 // position k of head i: row i, 16-byte unit k / 8 XOR-ed with i % 8
                 const int k = quad * 32 + lane;
-                uint8_t *pp = sm + L.p + (j & 1) * 2 * NH * 128 + group * HH * 128 + (k & 7) * 2;
+                uint8_t *pp = sm + L.p + (j & 1) * 2 * NH * 128 + group * HH * 128 + (k & 6) * 2;
+                const bool odd = (lane & 1) != 0;
+                uint32_t both[HH];                           // high term, low term
 #pragma unroll
                 for (int i = 0; i < HH; ++i) {
                     const float e = ex2(s[i] - w_m[i]);
                     v[i] = e;
-                    const uint32_t hi = dense::bf16_pair(e, 0.0f);
-                    uint8_t *at = pp + i * 128 + (((k >> 3) ^ (i & 7)) << 4);
-                    *reinterpret_cast<uint16_t *>(at) = static_cast<uint16_t>(hi);
-                    *reinterpret_cast<uint16_t *>(at + NH * 128) = dense::f32_bf16(e - __uint_as_float(hi << 16));
+                    const float hi = __uint_as_float(dense::bf16_pair(e, 0.0f) << 16);
+                    both[i] = dense::bf16_pair(hi, e - hi);
+                }
+                // neighbouring lanes hold neighbouring positions: one writes both of head i, the other both of head i + 1
+#pragma unroll
+                for (int i = 0; i < HH; i += 2) {
+                    const uint32_t got = __shfl_xor_sync(0xffffffffu, odd ? both[i] : both[i + 1], 1), own = odd ? both[i + 1] : both[i];
+                    const uint32_t first = odd ? got : own, second = odd ? own : got;
+                    const int head = i + (odd ? 1 : 0);
+                    uint8_t *at = pp + head * 128 + (((k >> 3) ^ (head & 7)) << 4);
+                    *reinterpret_cast<uint32_t *>(at) = __byte_perm(first, second, 0x5410);
+                    *reinterpret_cast<uint32_t *>(at + NH * 128) = __byte_perm(first, second, 0x7632);
                 }
                 l = l * corr + over_lanes<HH, false>(v, lane);
                 if (key >= total && group == 0) {             // nothing has been written there: its weight is zero, but the bits must be numbers

@@ -705,6 +705,56 @@ __global__ void __launch_bounds__(512) gated_norm_block_kernel(const GatedParams
     for (int i = threadIdx.x; i < p.group; i += 512) dense::put(out + i, o[i] * r * p.w[i] * dense::sigmoid(dense::get(gate + i)));
 }
 
+__device__ __forceinline__ float4 get4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 get4(const uint16_t *p) {
+    const uint2 b = *reinterpret_cast<const uint2 *>(p);
+    return make_float4(__uint_as_float(b.x << 16), __uint_as_float(b.x & 0xffff0000u), __uint_as_float(b.y << 16), __uint_as_float(b.y & 0xffff0000u));
+}
+__device__ __forceinline__ float gate_of(const float *, float z) { return dense::sigmoid(z); }
+__device__ __forceinline__ float gate_of(const uint16_t *, float z) { return __frcp_rn(1.0f + __expf(-z)); }
+// The same with four neighbouring values a thread, held in registers between the sum and the product: a block (LANES = 256)
+// or a warp (32, eight groups a block) per group of up to 4 LANES NV values.
+template <typename T, int LANES, int NV>
+__global__ void __launch_bounds__(256) gated_norm_vec_kernel(const GatedParams p) {
+    ptx::pdl_trigger();
+    ptx::pdl_wait();
+    __shared__ float s_red[32];
+    const int lane = threadIdx.x % LANES, g = blockIdx.x * (256 / LANES) + threadIdx.x / LANES, n4 = p.group >> 2;
+    const size_t row = blockIdx.y, at = static_cast<size_t>(g) * p.group;
+    if (LANES == 32 && at >= static_cast<size_t>(p.n)) return;
+    const float *o = p.o + row * p.n + at;
+    const T *gate = static_cast<const T *>(p.gate) + row * p.ldg + at;
+    float4 v[NV], z[NV];
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int i = lane + j * LANES;
+        v[j] = z[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n4) {
+            v[j] = get4(o + 4 * i);
+            z[j] = get4(gate + 4 * i);
+        }
+        ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+    }
+    if (LANES == 32) {
+#pragma unroll
+        for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+    } else {
+        ss = dense::block_sum<256>(ss, s_red);
+    }
+    const float r = 1.0f / sqrtf(ss / static_cast<float>(p.group) + p.eps);
+    T *out = static_cast<T *>(p.out) + row * p.ldo + at;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int i = lane + j * LANES;
+        if (i < n4) {
+            const float4 w = __ldg(reinterpret_cast<const float4 *>(p.w) + i);
+            dense::put4(out + 4 * i, make_float4(v[j].x * r * w.x * gate_of(gate, z[j].x), v[j].y * r * w.y * gate_of(gate, z[j].y), v[j].z * r * w.z * gate_of(gate, z[j].z),
+                                                 v[j].w * r * w.w * gate_of(gate, z[j].w)));
+        }
+    }
+}
+
 constexpr size_t kRingBytes = 128 * 1024;  // two records of the largest sizes fit
 
 template <typename T, bool DELTA>
@@ -854,6 +904,19 @@ int launch_gated_norm(Ctx *ctx, const GatedNormCall &c, cudaStream_t st) {
     GatedParams p{c.o, c.w, c.gate, c.out, c.ldg, c.ldo, static_cast<int>(c.n), static_cast<int>(c.group), c.eps};
     const bool f32 = c.compute == LBK_COMPUTE_F32;
     const unsigned groups = static_cast<unsigned>(c.n / c.group), rows = static_cast<unsigned>(c.rows);
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(c.o) | reinterpret_cast<uintptr_t>(c.w) | reinterpret_cast<uintptr_t>(c.gate) | reinterpret_cast<uintptr_t>(c.out);
+    if (c.group % 4 == 0 && c.ldg % 4 == 0 && c.ldo % 4 == 0 && (bits & 15) == 0 && c.group <= 8192) {
+        void (*k)(GatedParams);
+        const bool warp = c.group <= 256;
+        if (warp) k = f32 ? gated_norm_vec_kernel<float, 32, 2> : gated_norm_vec_kernel<uint16_t, 32, 2>;
+        else if (c.group <= 1024) k = f32 ? gated_norm_vec_kernel<float, 256, 1> : gated_norm_vec_kernel<uint16_t, 256, 1>;
+        else if (c.group <= 4096) k = f32 ? gated_norm_vec_kernel<float, 256, 4> : gated_norm_vec_kernel<uint16_t, 256, 4>;
+        else k = f32 ? gated_norm_vec_kernel<float, 256, 8> : gated_norm_vec_kernel<uint16_t, 256, 8>;
+        LBK_CUDA(launch_chained(k, dim3(warp ? (groups + 7) / 8 : groups, rows), dim3(256), 0, st, p));
+        LBK_CUDA(cudaGetLastError());
+        ctx->launches++;
+        return LBK_OK;
+    }
     if (c.group <= 256) LBK_CUDA(launch_chained(f32 ? gated_norm_warp_kernel<float> : gated_norm_warp_kernel<uint16_t>, dim3((groups + 7) / 8, rows), dim3(256), 0, st, p));
     else LBK_CUDA(launch_chained(f32 ? gated_norm_block_kernel<float> : gated_norm_block_kernel<uint16_t>, dim3(groups, rows), dim3(512), 0, st, p));
     LBK_CUDA(cudaGetLastError());
