@@ -60,7 +60,7 @@ def make_config(vocab: int, width: int, layers: list, eps: float = 1e-6) -> dict
     return {"architecture": ARCHITECTURE, "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
 
 
-def tensor_shapes(cfg: dict, low_rank: int = 24) -> Iterator[Tuple[str, Tuple[int, ...]]]:
+def tensor_shapes(cfg: dict, low_rank: int = 16) -> Iterator[Tuple[str, Tuple[int, ...]]]:
     """(name, shape) of every tensor of a model, in file order. low_rank: inner size of the delta rule's two-step
     projections, which the configuration does not fix."""
     V, W = cfg["vocab"], cfg["width"]
@@ -107,7 +107,7 @@ def tensor_shapes(cfg: dict, low_rank: int = 24) -> Iterator[Tuple[str, Tuple[in
     yield "final.norm", (W,)
 
 
-def random_checkpoint(cfg: dict, seed: int = 0, low_rank: int = 24) -> Dict[str, np.ndarray]:
+def random_checkpoint(cfg: dict, seed: int = 0, low_rank: int = 16) -> Dict[str, np.ndarray]:
     """Random weights as bf16 bits: matrices N(0, 1 / columns), embedding N(0, 1), norm weights near their neutral value,
     decays of the delta rule between none and strong."""
     rng = np.random.default_rng(seed)
