@@ -583,11 +583,7 @@ __global__ void __launch_bounds__(kGThreads, 1) dense_gemm_kernel(const __grid_c
                 } else {
                     tmem_ld_wait();
                 }
-                if (plan.mode) {
-#pragma unroll
-                    for (int i = 0; i < 32; ++i)
-                        if (c * 32 + i < ntok) dense::row_store<uint16_t>(p.epi, plan, tok0 + c * 32 + i, __uint_as_float(v[i]));
-                }
+                dense::row_store_run<uint16_t>(p.epi, plan, tok0 + c * 32, ntok - c * 32, v);
             }
             tc_fence_before();
             __syncwarp();

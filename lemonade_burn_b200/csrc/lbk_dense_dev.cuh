@@ -61,7 +61,7 @@ __device__ __forceinline__ float block_sum(float v, float *s_red) {
 
 // Where output row r of a call goes, worked out once per row; the token is added per store.
 struct RowPlan {
-    int mode = 0;  // 0: drop, 1: f32, 2: compute type with the activation, 3: compute type
+    int mode = 0;  // 0: drop, 1: f32, 2: compute type with squared relu, 3: compute type, 4: with silu
     float bias = 0.0f;
     char *base = nullptr;
     long stride = 0, seq_stride = 0;
@@ -81,7 +81,7 @@ __device__ __forceinline__ RowPlan row_plan(const DenseEpi &e, int r, int pos0) 
             q.base = reinterpret_cast<char *>(e.out2 + (r - e.f32_from));
             q.stride = e.ld2;
         } else {
-            q.mode = r < e.act_rows ? 2 : 3;
+            q.mode = r >= e.act_rows || e.act == kActNone ? 3 : e.act == kActRelu2 ? 2 : 4;
             q.base = reinterpret_cast<char *>(static_cast<T *>(e.out) + r);
             q.stride = e.ld;
         }
@@ -122,8 +122,40 @@ __device__ __forceinline__ void row_store(const DenseEpi &e, const RowPlan &q, i
     }
     v += q.bias;
     if (q.mode == 1) reinterpret_cast<float *>(q.base)[off] = v;
-    else if (q.mode == 2) put(reinterpret_cast<T *>(q.base) + off, e.act == kActRelu2 ? relu2(v) : e.act == kActSilu ? silu<sizeof(T) == 4>(v) : v);
-    else if (q.mode == 3) put(reinterpret_cast<T *>(q.base) + off, v);
+    else if (q.mode) put(reinterpret_cast<T *>(q.base) + off, q.mode == 3 ? v : q.mode == 2 ? relu2(v) : silu<sizeof(T) == 4>(v));
+}
+// Tokens t0 .. t0 + min(N, cnt) - 1 of one row at once, the choice of what to do with them outside the loop.
+template <typename T, int N>
+__device__ __forceinline__ void row_store_run(const DenseEpi &e, const RowPlan &q, int t0, int cnt, const uint32_t (&v)[N]) {
+    if (q.mode == 0) return;
+    if (q.by_pos) {
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            if (i < cnt) row_store<T>(e, q, t0 + i, __uint_as_float(v[i]));
+        return;
+    }
+    const long first = static_cast<long>(t0) * q.stride;
+    if (q.mode == 1) {
+        float *o = reinterpret_cast<float *>(q.base) + first;
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            if (i < cnt) o[i * q.stride] = __uint_as_float(v[i]) + q.bias;
+        return;
+    }
+    T *o = reinterpret_cast<T *>(q.base) + first;
+    if (q.mode == 2) {
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            if (i < cnt) put(o + i * q.stride, relu2(__uint_as_float(v[i]) + q.bias));
+    } else if (q.mode == 4) {
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            if (i < cnt) put(o + i * q.stride, silu<sizeof(T) == 4>(__uint_as_float(v[i]) + q.bias));
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            if (i < cnt) put(o + i * q.stride, __uint_as_float(v[i]) + q.bias);
+    }
 }
 // A prompt pass whose positions do not fit the cache must not store anything.
 __device__ __forceinline__ bool rows_fit(const DenseEpi &e, int m, int &pos0) {
