@@ -38,11 +38,11 @@ __device__ __forceinline__ float relu2(float z) {
     return r * r;
 }
 
-// z / (1 + e^-z); e^-z overflows to inf for large negative z: -0
+// z / (1 + e^-z); e^-z overflows to inf for large negative z: 0, as it should be
 template <bool EXACT>
 __device__ __forceinline__ float silu(float z) {
     if (EXACT) return z / (1.0f + expf(-z));
-    return z * __frcp_rn(1.0f + __expf(-z));
+    return __fdividef(z, 1.0f + __expf(-z));
 }
 
 // Sum over the block; every thread gets it. `s_red`: 32 floats, may be reused right away.

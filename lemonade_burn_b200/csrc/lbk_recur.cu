@@ -711,7 +711,7 @@ __device__ __forceinline__ float4 get4(const uint16_t *p) {
     return make_float4(__uint_as_float(b.x << 16), __uint_as_float(b.x & 0xffff0000u), __uint_as_float(b.y << 16), __uint_as_float(b.y & 0xffff0000u));
 }
 __device__ __forceinline__ float gate_of(const float *, float z) { return dense::sigmoid(z); }
-__device__ __forceinline__ float gate_of(const uint16_t *, float z) { return __frcp_rn(1.0f + __expf(-z)); }
+__device__ __forceinline__ float gate_of(const uint16_t *, float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 // The same with four neighbouring values a thread, held in registers between the sum and the product: a block (LANES = 256)
 // or a warp (32, eight groups a block) per group of up to 4 LANES NV values.
 template <typename T, int LANES, int NV>
